@@ -40,6 +40,9 @@ EXPORTED_SYMBOLS = [
     "gptb200_embedding_decode", "gptb200_kv_cache_fill", "gptb200_attention_decode", "gptb200_advance_position",
     "gptb200_loader_create", "gptb200_loader_destroy", "gptb200_loader_num_samples", "gptb200_loader_reset_epoch", "gptb200_loader_next_batch",
     "gptb200_bias_grad_noalloc",
+    "gptb200_decoder_check_config", "gptb200_decoder_load", "gptb200_decoder_destroy", "gptb200_decoder_context", "gptb200_decoder_vocab",
+    "gptb200_decoder_open", "gptb200_decoder_close", "gptb200_decoder_length", "gptb200_decoder_set_option", "gptb200_decoder_step",
+    "gptb200_decoder_generate", "gptb200_rotary_frequencies", "gptb200_sample_rows",
 ]
 
 

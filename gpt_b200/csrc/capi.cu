@@ -16,6 +16,7 @@
 #include "gemm_sm100.cuh"
 #include "gemm_sm100_pair.cuh"
 #include "skinny_sm100.cuh"
+#include "gemv_bf16.cuh"
 #include "kernels_misc.cuh"
 
 using namespace gptb200;
@@ -141,6 +142,7 @@ struct GemmCall {
     bool accumulate;  // out += result
     float *dbias = nullptr;  // grad_w form only: dbias[N] += column sums of b, inside the same launch when the CTA-pair kernel runs
     const float *gelu_src = nullptr;  // out = result * gelu_tanh'(gelu_src) element by element, when the CTA-pair kernel runs
+    bool fma_only = false;            // fp32 FMAs whatever the mode
 };
 
 template <int BN, bool A_MN, bool B_MN, bool X3>
@@ -437,7 +439,9 @@ int run_gemm(gptb200_ctx *ctx, const GemmCall &c, bool *dbias_fused = nullptr, b
 {
     if (dbias_fused) *dbias_fused = false;
     if (gelu_fused) *gelu_fused = false;
-    const GemmPlan pl = plan_gemm(plan_input(ctx, c));
+    GemmPlanInput in = plan_input(ctx, c);
+    in.fma_only = c.fma_only;
+    const GemmPlan pl = plan_gemm(in);
     if (pl.kernel == KERNEL_NONE) return GPTB200_OK;
     if (pl.kernel == KERNEL_SKINNY) return run_skinny(ctx, c, pl);
     if (pl.kernel == KERNEL_SIMT) {
@@ -678,6 +682,135 @@ int run_gemm_batched_impl(gptb200_ctx *ctx, float *out, long long out_ld, long l
     return GPTB200_OK;
 }
 
+// 2-D tensor map of 4-byte words with a row pitch: bf16 operands (box 32 words x box_rows, 128-byte swizzle) and 16-bit outputs
+// (box 16 words x 32 rows, 64-byte swizzle; the map is 3-D because the stores are).
+int make_word_tmap(gptb200_ctx *ctx, CUtensorMap *map, const void *base, long long rows, long long words, long long pitch, int box_words, int box_rows, bool output)
+{
+    const TmapKey key{reinterpret_cast<uintptr_t>(base), words, rows, pitch, box_words, box_rows, output ? 7 : 6};
+    const auto hit = ctx->tmaps.find(key);
+    if (hit != ctx->tmaps.end()) {
+        *map = hit->second;
+        return GPTB200_OK;
+    }
+    cuuint64_t dims[3] = {static_cast<cuuint64_t>(words), static_cast<cuuint64_t>(rows), 1};
+    cuuint64_t strides[2] = {static_cast<cuuint64_t>(pitch) * 4, static_cast<cuuint64_t>(pitch) * 4 * rows};
+    cuuint32_t box[3] = {static_cast<cuuint32_t>(box_words), static_cast<cuuint32_t>(box_rows), 1};
+    cuuint32_t estr[3] = {1, 1, 1};
+    const CUresult r = ctx->encode(map, CU_TENSOR_MAP_DATA_TYPE_UINT32, output ? 3 : 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                                   box_words == 16 ? CU_TENSOR_MAP_SWIZZLE_64B : CU_TENSOR_MAP_SWIZZLE_128B,
+                                   output ? CU_TENSOR_MAP_L2_PROMOTION_NONE : CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    ctx->tmap_encodes++;
+    if (r != CUDA_SUCCESS)
+        return fail(ctx, GPTB200_ERR_CUDA, "cuTensorMapEncodeTiled (16-bit) failed (%d) rows=%lld words=%lld pitch=%lld", int(r), rows, words, pitch);
+    if (ctx->tmaps.size() >= kTmapCacheMax) ctx->tmaps.clear();
+    ctx->tmaps.emplace(key, *map);
+    return GPTB200_OK;
+}
+
+template <int MR>
+int launch_gemv(gptb200_ctx *ctx, const GemvParams &g)
+{
+    const size_t smem = size_t(MR) * g.K * 2;
+    auto kernel = gemv_bf16_kernel<MR>;
+    const void *key = reinterpret_cast<const void *>(kernel);
+    if (smem > 48 * 1024 && !ctx->configured.count(key)) {
+        CUDA_TRY(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        ctx->configured.insert(key);
+    }
+    const int pairs = g.out_kind == OUT_GLU ? g.N / 2 : (g.N + 1) / 2;
+    const int per_cta = kGemvThreads / 32;
+    const int ctas = std::max(1, std::min((pairs + per_cta - 1) / per_cta, ctx->num_sms * 4));
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3(ctas);
+    cfg.blockDim = dim3(kGemvThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    cudaLaunchAttribute attr{};
+    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr.val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = &attr;
+    cfg.numAttrs = ctx->decode_early_launch ? 1 : 0;
+    ctx->launches++;
+    CUDA_TRY(ctx, cudaLaunchKernelEx(&cfg, kernel, g));
+    return GPTB200_OK;
+}
+
+int run_linear_bf16_impl(gptb200_ctx *ctx, const Bf16Linear &c)
+{
+    if (c.M <= 0 || c.N <= 0) return GPTB200_OK;
+    if (c.K <= 0 || c.K % 8 || c.lda % 8 || !aligned16(c.a) || !aligned16(c.w) || !aligned16(c.out) || (c.out_kind == OUT_GLU && c.N % 64) ||
+        (c.out_kind == OUT_BF16 && c.tail_col % 32 && c.tail_col < c.N) || (c.out_kind == OUT_GELU_MUL && (c.N % 8 || c.factor_pitch % 8 || !aligned16(c.factor))))
+        return fail(ctx, GPTB200_ERR_INVALID_ARG, "bf16 product: sizes or alignment (M=%d N=%d K=%d lda=%lld kind=%d)", c.M, c.N, c.K, c.lda, c.out_kind);
+    if (c.M <= ctx->gemv_rows && size_t(c.M <= 1 ? 1 : c.M <= 2 ? 2 : c.M <= 4 ? 4 : 8) * c.K * 2 <= 200 * 1024) {
+        GemvParams g{c.M, c.N, c.K, static_cast<const uint16_t *>(c.a), c.lda, static_cast<const uint16_t *>(c.w), c.out_kind, c.out, c.ldo, c.tail, c.tail_col, c.tail_pitch,
+                     static_cast<const uint16_t *>(c.factor), c.factor_rows, c.factor_pitch};
+        return c.M <= 1 ? launch_gemv<1>(ctx, g) : c.M <= 2 ? launch_gemv<2>(ctx, g) : c.M <= 4 ? launch_gemv<4>(ctx, g) : launch_gemv<8>(ctx, g);
+    }
+    const bool f32 = c.out_kind == OUT_F32;
+    const long long out_words = f32 ? c.N : c.out_kind == OUT_GLU ? c.N / 4 : (std::min(c.N, c.tail_col) + 1) / 2;
+    const long long ldo_words = f32 ? c.ldo : c.ldo / 2;
+    if (ldo_words % 4 || c.ldo % 2) return fail(ctx, GPTB200_ERR_INVALID_ARG, "bf16 product: output pitch %lld", c.ldo);
+    GemmPlanInput in{};
+    in.M = c.M; in.N = (c.N + 3) & ~3; in.K = c.K / 2;      // in 4-byte words: a k-block of 32 words is 64 bf16
+    in.has_epilogue = !f32 || c.ldo != c.N || c.N % 4 != 0;   // split-K adds contiguous fp32 partial sums
+    in.aligned = true;
+    in.num_sms = ctx->max_sms > 0 ? std::min(ctx->max_sms, ctx->num_sms) : ctx->num_sms;
+    in.opt_tile_n = ctx->tile_n; in.opt_max_splits = ctx->max_splits; in.opt_pair = ctx->pair; in.opt_stream_k = ctx->stream_k;
+    in.ws_limit = ctx->ws_limit;
+    const GemmPlan pl = plan_gemm(in);
+    const bool pair = pl.kernel == KERNEL_PAIR;
+    if (!pair && pl.kernel != KERNEL_SINGLE) return fail(ctx, GPTB200_ERR_INVALID_ARG, "bf16 product: no kernel for M=%d N=%d K=%d", c.M, c.N, c.K);
+    GemmParams p{};
+    p.M = c.M; p.N = c.N; p.K = in.K;
+    p.tiles_m = pl.tiles_m; p.tiles_n = pl.tiles_n; p.num_kb = pl.num_kb; p.kb_per_split = pl.kb_per_split; p.splits = pl.splits;
+    p.status = ctx->d_status;
+    p.bf16 = 1;
+    p.out_kind = c.out_kind;
+    p.tail = c.tail; p.tail_col = c.tail_col; p.tail_pitch = c.tail_pitch;
+    p.factor = c.factor; p.factor_rows = c.factor_rows; p.factor_pitch = c.factor_pitch;
+    p.epi_mode = EPI_STORE;
+    float *out_base = static_cast<float *>(c.out);
+    if (pair) {
+        p.sk_total = pl.sk_total;
+        p.sk_unit = pl.sk_unit;
+        if (pl.sk_max_share > 1) {
+            const int rc = ensure_workspace(ctx, pl.workspace_bytes);
+            if (rc != GPTB200_OK) return rc;
+            p.sk_slots = ctx->ws;
+            p.sk_flags = ctx->d_pair_flags;
+            p.sk_state = ctx->d_pair_flags + size_t(ctx->num_sms) * 8;
+        }
+    } else if (pl.splits > 1) {
+        const int rc = ensure_workspace(ctx, size_t(c.M) * c.N * sizeof(float) * pl.splits);
+        if (rc != GPTB200_OK) return rc;
+        out_base = ctx->ws;
+        p.epi_mode = EPI_PARTIAL;
+    }
+    CUtensorMap ta, tb, to;
+    int rc = make_word_tmap(ctx, &ta, c.a, c.M, c.K / 2, c.lda / 2, kBK, kBM, false);
+    if (rc == GPTB200_OK) rc = make_word_tmap(ctx, &tb, c.w, c.N, c.K / 2, c.K / 2, kBK, pair ? pl.tile_n / 2 : pl.tile_n, false);
+    if (rc == GPTB200_OK && pl.splits > 1) rc = make_out_tmap(ctx, &to, out_base, pl.splits, c.M, c.N);
+    if (rc == GPTB200_OK && pl.splits <= 1) rc = make_word_tmap(ctx, &to, c.out, c.M, out_words, ldo_words, f32 ? 32 : 16, 32, true);
+    if (rc != GPTB200_OK) return rc;
+    cudaError_t e;
+    if (pair)
+        e = launch_pair_instance<false, false, false>(ctx, ta, tb, to, to, to, p, pl.grid);
+    else if (pl.tile_n == 256)
+        e = launch_instance<256, false, false, false>(ctx, ta, tb, to, to, p, pl.grid);
+    else
+        e = launch_instance<128, false, false, false>(ctx, ta, tb, to, to, p, pl.grid);
+    ctx->launches++;
+    CUDA_TRY(ctx, e);
+    if (pl.splits > 1) {
+        const long long n4 = (1LL * c.M * c.N) >> 2;
+        const int blocks = static_cast<int>(std::min<long long>((n4 + 255) / 256, 1LL * ctx->num_sms * 8));
+        splitk_reduce_kernel<<<blocks, 256, 0, ctx->stream>>>(static_cast<float *>(c.out), ctx->ws, n4, pl.splits, 0);
+        ctx->launches++;
+        CUDA_TRY(ctx, cudaGetLastError());
+    }
+    return GPTB200_OK;
+}
+
 int check_dims(gptb200_ctx *ctx, int m, int a, int b)
 {
     if (!ctx) return GPTB200_ERR_INVALID_ARG;
@@ -695,6 +828,15 @@ int run_gemm_batched(gptb200_ctx *ctx, float *out, long long out_ld, long long o
                      int M, int N, int K, int inner, int outer, bool causal)
 {
     return run_gemm_batched_impl(ctx, out, out_ld, out_si, out_so, a, b, M, N, K, inner, outer, causal);
+}
+
+int run_linear_bf16(gptb200_ctx *ctx, const Bf16Linear &c) { return run_linear_bf16_impl(ctx, c); }
+
+int run_linear_f32(gptb200_ctx *ctx, float *out, const float *a, const float *w, int M, int N, int K)
+{
+    GemmCall c{M, N, K, a, false, w, false, out, nullptr, nullptr, false};
+    c.fma_only = true;
+    return run_gemm(ctx, c);
 }
 }  // namespace gptb200
 

@@ -58,6 +58,7 @@ struct gptb200_ctx {
     int skinny_cluster_rows = 8;   // ... for calls with at most this many rows
     int skinny_tile_rows = 0;      // that kernel's row tile beyond 32 rows: 0 or 64 = one tile of 64, 32 = row groups of 32
     bool skinny_tile = true;       // beyond that many rows: one-launch register-tiled cluster kernel (false: the k-split kernel)
+    int gemv_rows = 8;             // bf16 products: most rows the weight-streaming kernel takes (0 .. 8)
     int decode_early_launch = 0;     // that kernel is launched with programmatic stream serialization: it prefetches weights while
                                        // its predecessor on the stream still runs (caller's promise: the predecessor does not write them)
     bool skinny_rowwise = true;  // W stored [n][k], no bias: one-launch warp-per-row kernel ...
@@ -121,6 +122,27 @@ struct BatchedOperand {
 // causal: the consumer of a square product reads only columns <= row, so output pieces wholly beyond the diagonal may stay unwritten
 int run_gemm_batched(gptb200_ctx *ctx, float *out, long long out_ld, long long out_si, long long out_so, const BatchedOperand &a, const BatchedOperand &b,
                      int M, int N, int K, int inner, int outer, bool causal = false);
+
+// out[m][n] = a[m][k] . w[n][k] with bf16 operands and fp32 accumulation (capi.cu): the tensor-core kernels for more than
+// eight rows, a weight-streaming kernel below.  K and the pitches are multiples of 8 elements, bases 16-byte aligned.
+struct Bf16Linear {
+    int M, N, K;
+    const void *a;              // bf16, row pitch lda
+    long long lda;
+    const void *w;              // bf16 [N][K]
+    int out_kind;               // OutKind (gemm_sm100.cuh)
+    void *out;                  // fp32 or bf16, row pitch ldo in elements
+    long long ldo;
+    float *tail = nullptr;      // OUT_BF16: columns from tail_col (a multiple of 32) on stay fp32
+    int tail_col = 0x7fffffff, tail_pitch = 0;
+    const void *factor = nullptr;   // OUT_GELU_MUL
+    const int *factor_rows = nullptr;
+    int factor_pitch = 0;
+};
+int run_linear_bf16(gptb200_ctx *ctx, const Bf16Linear &c);
+
+// out[m][n] = a[m][k] . w[n][k] in fp32 FMAs only (no tensor core), whatever the context's mode.
+int run_linear_f32(gptb200_ctx *ctx, float *out, const float *a, const float *w, int M, int N, int K);
 
 // Grows the context's scratch buffer to at least `bytes` (waits for queued work before replacing it).
 int ensure_workspace(gptb200_ctx *ctx, size_t bytes);

@@ -30,6 +30,7 @@ struct GemmPlanInput {
     bool opt_skinny;
     int opt_skinny_rows;     // most rows the weight-streaming kernel takes; 0 = kPlanSkinnyMaxRows
     size_t ws_limit;         // scratch limit in bytes
+    bool fma_only;           // fp32 FMAs only: no tensor-core kernel
 };
 
 struct GemmPlan {
@@ -187,7 +188,7 @@ inline GemmPlan plan_gemm(const GemmPlanInput &in)
     const long long lda = in.a_mn ? in.M : in.K;
     const long long ldb = in.b_mn ? in.N : in.K;
     const bool tma_ok = in.K > 0 && in.aligned && lda % 4 == 0 && ldb % 4 == 0 && in.N % 4 == 0 && !(in.a_mn && !in.b_mn);
-    if (!tma_ok) {
+    if (!tma_ok || in.fma_only) {
         p.kernel = KERNEL_SIMT;
         p.tiles_m = (in.M + 31) / 32;
         p.tiles_n = (in.N + 31) / 32;

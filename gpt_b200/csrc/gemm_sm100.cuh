@@ -54,6 +54,14 @@ enum EpilogueMode : int {
     EPI_PARTIAL = 2,  // workspace[split] = acc   (reduced by splitk_reduce_kernel)
 };
 
+// Outputs of the bf16 form (GemmParams::bf16).
+enum OutKind : int {
+    OUT_F32 = 0,        // fp32 through the output tensor map, like the other forms
+    OUT_BF16 = 1,       // rounded to bf16; columns from tail_col on stay fp32 and go to `tail`
+    OUT_GLU = 2,        // columns come in groups of 32 gate | 32 up: gelu_tanh(gate) * up in bf16, half as many columns
+    OUT_GELU_MUL = 3,   // gelu_tanh(out) * factor[factor_rows[row]][column] in bf16
+};
+
 struct GemmParams {
     int M, N, K;         // D[M x N] = A[M x K] . B[K x N]
     const float *bias;   // optional [N]
@@ -106,6 +114,15 @@ struct GemmParams {
     int dbias_rows;          // tile rows that share the column sums (1: the first tile row does them all)
     float *dbias_part;       // [tile row][tiles_n * 256] the tiles' shares
     unsigned int *dbias_tickets;   // [tile column][CTA][epilogue warp] shares parked so far (reset by the last one)
+    // bf16 form (both operands K-major, not 3xTF32): a k-block is 64 bf16 values, the same 128-byte rows and the same swizzled tiles as
+    // 32 floats, so producer, ring and descriptors are those of the TF32 form and only the instruction differs.  K counts 4-byte words.
+    int bf16;
+    int out_kind;               // OutKind; the 16-bit kinds are staged as [32 rows x 64 bytes] and stored through tmap_act
+    float *tail;                // OUT_BF16: fp32 columns [M][tail_pitch]
+    int tail_col, tail_pitch;   // first of them (a multiple of 32; >= N: none)
+    const void *factor;         // OUT_GELU_MUL: bf16 table, row pitch factor_pitch (a multiple of 8), 16-byte aligned
+    const int *factor_rows;     // row of the table per output row
+    int factor_pitch;
 };
 
 constexpr int kTraceSlots = 128;
@@ -190,6 +207,61 @@ __device__ __forceinline__ float gelu_tanh_grad_fast(float x)
     const float u = 0.79788456f * (x + 0.044715f * x * x * x);
     const float t = 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * u));
     return 0.5f * (1.0f + t) + 0.5f * x * (1.0f - t * t) * (0.79788456f + 0.107032f * x * x);
+}
+
+__device__ __forceinline__ float bf16_lo(uint32_t w) { return __uint_as_float(w << 16); }
+__device__ __forceinline__ float bf16_hi(uint32_t w) { return __uint_as_float(w & 0xFFFF0000u); }
+
+// One [32 rows x 32 columns] piece of a 16-bit output (this thread: row row0 + lane).  Returns false when there is nothing to stage;
+// otherwise `w` holds the row's 32 bf16 values and `word0` the first 4-byte word of the piece in the output row.  `held`
+// carries the gate columns of OUT_GLU from one piece to the next.
+__device__ __forceinline__ bool piece_to_bf16(const GemmParams &p, float (&v)[32], float (&held)[32], int row0, int col0, int lane, uint32_t (&w)[16], int &word0)
+{
+    word0 = col0 / 2;
+    if (p.out_kind == OUT_BF16) {
+        if (col0 >= p.tail_col) {
+            if (row0 + lane < p.M) {
+                float *dst = p.tail + static_cast<long long>(row0 + lane) * p.tail_pitch + (col0 - p.tail_col);
+#pragma unroll
+                for (int j = 0; j < 32; ++j)
+                    if (col0 + j < p.N) dst[j] = v[j];
+            }
+            return false;
+        }
+    } else if (p.out_kind == OUT_GLU) {
+        if (!(col0 & 32)) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) held[j] = v[j];
+            return false;
+        }
+        word0 = (col0 - 32) / 4;
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[j] *= gelu_tanh(held[j]);
+    } else {
+        const bool row_ok = row0 + lane < p.M;
+        const uint4 *f = reinterpret_cast<const uint4 *>(static_cast<const uint16_t *>(p.factor) +
+                                                         (row_ok ? static_cast<long long>(p.factor_rows[row0 + lane]) * p.factor_pitch : 0) + col0);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+            const uint4 t = row_ok && col0 + 8 * q < p.N ? __ldg(f + q) : make_uint4(0u, 0u, 0u, 0u);   // N is a multiple of 8
+            const uint32_t x[4] = {t.x, t.y, t.z, t.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                v[8 * q + 2 * e] = gelu_tanh(v[8 * q + 2 * e]) * bf16_lo(x[e]);
+                v[8 * q + 2 * e + 1] = gelu_tanh(v[8 * q + 2 * e + 1]) * bf16_hi(x[e]);
+            }
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < 16; ++j) w[j] = ptx::pack_bf16x2(v[2 * j], v[2 * j + 1]);
+    return row0 < p.M && col0 < p.N;
+}
+
+// Writes this thread's 16 words (row = lane) into a [32 rows x 64 bytes] staging tile with the 64-byte swizzle of its tensor map.
+__device__ __forceinline__ void stage_row_bf16(uint32_t buf, int lane, const uint32_t (&w)[16])
+{
+#pragma unroll
+    for (int j = 0; j < 4; ++j) ptx::sts128(buf + lane * 64 + ((j ^ ((lane >> 1) & 3)) << 4), w[4 * j], w[4 * j + 1], w[4 * j + 2], w[4 * j + 3]);
 }
 
 // One epilogue warp's staging state: `kBufs` swizzled [32 x 32] fp32 tiles and the count of TMA stores
@@ -391,6 +463,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
                                     ptx::mma_tf32_ss(d_tmem, da_lo, db_hi, kIdesc, accumulate);
                                     ptx::mma_tf32_ss(d_tmem, da_hi, db_lo, kIdesc, 1u);
                                     ptx::mma_tf32_ss(d_tmem, da_hi, db_hi, kIdesc, 1u);
+                                } else if (!A_MN && !B_MN && p.bf16) {
+                                    ptx::mma_f16_ss(d_tmem, da_hi, db_hi, ptx::make_idesc_bf16(kBM, BN, false, false), accumulate);
                                 } else {
                                     ptx::mma_tf32_ss(d_tmem, da_hi, db_hi, kIdesc, accumulate);
                                 }
@@ -423,8 +497,28 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
         uint32_t g = 0;
         bool ok = true;
 
+        float held[32];   // gate columns of OUT_GLU
         // bias / GELU, staging, TMA store of one [32 rows x 32 cols] piece of the tile
         auto emit = [&](float (&v)[32], int row0, int col0, int split) {
+            if constexpr (!A_MN && !B_MN && !X3) {
+                if (p.out_kind != OUT_F32 && p.epi_mode == EPI_STORE) {
+                    uint32_t w[16];
+                    int word0;
+                    const bool some = piece_to_bf16(p, v, held, row0, col0, lane, w, word0);
+                    if (__any_sync(0xffffffffu, some)) {
+                        const uint32_t buf = ring.acquire(lane);
+                        stage_row_bf16(buf, lane, w);
+                        ptx::fence_proxy_async_smem();
+                        __syncwarp();
+                        if (lane == 0) {
+                            ptx::tma_store_3d(&tmap_act, word0, row0, 0, buf);
+                            ptx::tma_store_commit();
+                        }
+                        ring.count++;
+                    }
+                    return;
+                }
+            }
             if (p.bias && p.epi_mode == EPI_STORE) {
 #pragma unroll
                 for (int j = 0; j < 32; ++j) v[j] += (col0 + j < p.N) ? __ldg(p.bias + col0 + j) : 0.0f;
@@ -580,7 +674,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
 // Self-test of the bounded wait: one thread waits, with a short limit, on a barrier that nothing will ever signal.
 // The wait runs out, the status word receives DEV_TIMEOUT_SELFTEST and the kernel returns normally: exactly the path
 // a real kernel takes when an expected signal never comes.
-__global__ void wait_timeout_selftest_kernel(int *status, long long limit_cycles)
+static __global__ void wait_timeout_selftest_kernel(int *status, long long limit_cycles)
 {
     __shared__ __align__(8) unsigned long long bar_storage;
     __shared__ uint32_t abort_flag;
@@ -596,7 +690,7 @@ __global__ void wait_timeout_selftest_kernel(int *status, long long limit_cycles
 }
 
 // out[i] (+)= sum_s ws[s][i], fixed order s = 0..splits-1 (deterministic split-K reduction).
-__global__ void splitk_reduce_kernel(float *__restrict__ out, const float *__restrict__ ws, long long n4, int splits, int accumulate)
+static __global__ void splitk_reduce_kernel(float *__restrict__ out, const float *__restrict__ ws, long long n4, int splits, int accumulate)
 {
     const long long stride = 1LL * gridDim.x * blockDim.x;
     for (long long i = 1LL * blockIdx.x * blockDim.x + threadIdx.x; i < n4; i += stride) {

@@ -688,7 +688,10 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                                 const uint32_t b_off = B_MN ? k * 1024 : k * 32;
                                 const uint64_t da_hi = ptx::make_smem_desc(a_hi + a_off, a_lbo, a_sbo, a_lay);
                                 const uint64_t db_hi = ptx::make_smem_desc(b_hi + b_off, b_lbo, b_sbo, b_lay);
-                                ptx::mma_tf32_ss_pair(d_tmem, da_hi, db_hi, idesc, accumulate);
+                                if (!A_MN && !B_MN && !X3 && p.bf16)
+                                    ptx::mma_f16_ss_pair(d_tmem, da_hi, db_hi, idesc_corr, accumulate);
+                                else
+                                    ptx::mma_tf32_ss_pair(d_tmem, da_hi, db_hi, idesc, accumulate);
                                 accumulate = 1u;
                             }
                             // the stage is free in both CTAs once these MMAs have read it
@@ -727,8 +730,28 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
         const uint32_t leader_tmem_empty[2] = {ptx::map_to_cta(tmem_empty_bar(0), 0u), ptx::map_to_cta(tmem_empty_bar(1), 0u)};
 
         int ezi = 0, ezo = 0;   // batched form: batch coordinates of the tile being written
+        float held[32];   // bf16 form: gate columns of OUT_GLU
         // bias_lane: bias[col0 + lane], fetched when the tile was started
         auto emit = [&](float (&v)[32], int row0, int col0, float bias_lane) {
+            if constexpr (!A_MN && !B_MN && !X3) {
+                if (p.out_kind != OUT_F32) {
+                    uint32_t w[16];
+                    int word0;
+                    const bool some = piece_to_bf16(p, v, held, row0, col0, lane, w, word0);
+                    if (__any_sync(0xffffffffu, some)) {
+                        const uint32_t buf = ring.acquire(lane);
+                        stage_row_bf16(buf, lane, w);
+                        ptx::fence_proxy_async_smem();
+                        __syncwarp();
+                        if (lane == 0) {
+                            ptx::tma_store_3d(&tmap_act, word0, row0, 0, buf);
+                            ptx::tma_store_commit();
+                        }
+                        ring.count++;
+                    }
+                    return;
+                }
+            }
             if (p.mma_n && col0 >= p.mma_n) return;   // narrow batched form: these accumulator columns were not computed
             if (p.causal_skip && col0 > row0 + 31) return;   // nobody reads these
             if (p.bias && p.epi_mode == EPI_STORE) {

@@ -1,0 +1,133 @@
+// Mamba-2 (state-space duality) layers: short causal convolution, step sizes and decays, the recurrence, the gated norm.
+//
+// A layer's projection row is [z: inner | x: inner | B: groups * state | C: groups * state] in T, its step sizes [heads] in fp32.  In a
+// sequence's slot: the convolution's last inputs [2][taps - 1][channels] in T (two copies, see StepEntry::parity) and
+// the state [heads][state][vdim] in fp32.  Steps, decays, exponentials, states and their sums are fp32.
+#pragma once
+
+#include "decoder_rows.cuh"
+
+namespace gptb200 {
+namespace dec {
+
+struct MambaShape {
+    int heads, vdim, state, groups, taps, norm_groups;
+    int inner, channels;        // heads * vdim; inner + 2 * groups * state
+    size_t conv_state, ssm_state;   // offsets in the slot
+};
+
+// Convolution + silu of one channel per thread; blocks beyond the channels compute the step sizes and log-decays.
+// xbc [rows][ld_xbc] T; dt, log_decay [rows][heads].
+template <typename T>
+__global__ void mamba_conv_kernel(T *__restrict__ xbc, int ld_xbc, float *__restrict__ dt, float *__restrict__ log_decay, const T *__restrict__ proj, long long ld_proj,
+                                  const float *__restrict__ dt_raw, int ld_dt, const float *__restrict__ taps, const float *__restrict__ conv_b,
+                                  const float *__restrict__ dt_bias, const float *__restrict__ a_log, const MambaShape s, const StepEntry *__restrict__ entries,
+                                  const int *__restrict__ row_entry, int conv_blocks)
+{
+    grid_dependency_wait();
+    grid_dependency_launch();
+    const int row = blockIdx.y;
+    if (static_cast<int>(blockIdx.x) >= conv_blocks) {
+        const int h = (blockIdx.x - conv_blocks) * blockDim.x + threadIdx.x;
+        if (h < s.heads) {
+            const float step = softplus_f(dt_raw[static_cast<long long>(row) * ld_dt + h] + dt_bias[h]);
+            dt[static_cast<long long>(row) * s.heads + h] = step;
+            log_decay[static_cast<long long>(row) * s.heads + h] = -expf(a_log[h]) * step;
+        }
+        return;
+    }
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= s.channels) return;
+    const StepEntry e = entries[row_entry[row]];
+    const int back = s.taps - 1;
+    T *state = reinterpret_cast<T *>(e.slot + s.conv_state);
+    const T *old = state + static_cast<long long>(e.parity) * back * s.channels;
+    const T *in = proj + s.inner + c;
+    // input `k` steps before row r (k < taps); before the portion: the sequence's state
+    auto input = [&](int r, int k) {
+        const int i = r - e.row0 - k;
+        return i >= 0 ? in[static_cast<long long>(r - k) * ld_proj] : old[static_cast<long long>(back + i) * s.channels + c];
+    };
+    float acc = conv_b[c];
+    for (int k = s.taps - 1; k >= 0; --k) acc = fmaf(taps[c * s.taps + (back - k)], to_f(input(row, k)), acc);
+    xbc[static_cast<long long>(row) * ld_xbc + c] = from_f<T>(silu_f(acc));
+    if (row == e.row0 + e.count - 1) {
+        T *next = state + static_cast<long long>(e.parity ^ 1) * back * s.channels;
+        for (int k = 0; k < back; ++k) next[static_cast<long long>(back - 1 - k) * s.channels + c] = input(row, k);
+    }
+}
+
+// The recurrence token by token: one block per (head, entry), state in shared memory.  y [rows][inner] fp32.
+template <typename T>
+__global__ void mamba_scan_kernel(float *__restrict__ y, const T *__restrict__ xbc, int ld_xbc, const float *__restrict__ dt, const float *__restrict__ log_decay,
+                                  const float *__restrict__ d_skip, const MambaShape s, const StepEntry *__restrict__ entries)
+{
+    extern __shared__ float sm[];
+    const int P = s.vdim, N = s.state, h = blockIdx.x;
+    const StepEntry e = entries[blockIdx.y];
+    const int lanes = blockDim.x / P;            // threads that share a column (>= 1)
+    float *S = sm;                               // [N][P]
+    float *part = S + N * P;                     // [lanes][P]
+    float *bc = part + lanes * P;                // B [N] | C [N] | x [P]
+    grid_dependency_wait();
+    grid_dependency_launch();
+    float *state = reinterpret_cast<float *>(e.slot + s.ssm_state) + static_cast<long long>(h) * N * P;
+    for (int i = threadIdx.x; i < N * P; i += blockDim.x) S[i] = state[i];
+    const int g = h / (s.heads / s.groups);
+    const int p = threadIdx.x % P, q = threadIdx.x / P;
+    const bool busy = q < lanes;
+    for (int t = 0; t < e.count; ++t) {
+        const int row = e.row0 + t;
+        const T *src = xbc + static_cast<long long>(row) * ld_xbc;
+        __syncthreads();
+        for (int i = threadIdx.x; i < N; i += blockDim.x) {
+            bc[i] = to_f(src[s.inner + g * N + i]);
+            bc[N + i] = to_f(src[s.inner + s.groups * N + g * N + i]);
+        }
+        for (int i = threadIdx.x; i < P; i += blockDim.x) bc[2 * N + i] = to_f(src[h * P + i]);
+        __syncthreads();
+        const float step = dt[static_cast<long long>(row) * s.heads + h], keep = expf(log_decay[static_cast<long long>(row) * s.heads + h]);
+        if (busy) {
+            const float x = bc[2 * N + p];
+            float acc = 0.0f;
+            for (int n = q; n < N; n += lanes) {
+                const float v = fmaf(keep, S[n * P + p], step * bc[n] * x);
+                S[n * P + p] = v;
+                acc = fmaf(bc[N + n], v, acc);
+            }
+            part[q * P + p] = acc;
+        }
+        __syncthreads();
+        if (threadIdx.x < P) {
+            float acc = 0.0f;
+            for (int i = 0; i < lanes; ++i) acc += part[i * P + threadIdx.x];
+            y[static_cast<long long>(row) * s.inner + h * P + threadIdx.x] = fmaf(d_skip[h], bc[2 * N + threadIdx.x], acc);
+        }
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < N * P; i += blockDim.x) state[i] = S[i];
+}
+
+// y * silu(z), then each of norm_groups parts divided by its own root mean square, times weight, as T [rows][ld_out].
+template <typename T>
+__global__ void mamba_gated_norm_kernel(T *__restrict__ out, int ld_out, const float *__restrict__ y, const T *__restrict__ proj, long long ld_proj,
+                                        const float *__restrict__ weight, const MambaShape s, float eps)
+{
+    extern __shared__ float sm[];   // [part]
+    __shared__ float red[32];
+    grid_dependency_wait();
+    grid_dependency_launch();
+    const long long row = blockIdx.x;
+    const int part = s.inner / s.norm_groups, c0 = blockIdx.y * part;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < part; i += blockDim.x) {
+        const float v = y[row * s.inner + c0 + i] * silu_f(to_f(proj[row * ld_proj + c0 + i]));
+        sm[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    const float inv = rsqrtf(block_sum(ss, red) / part + eps);
+    for (int i = threadIdx.x; i < part; i += blockDim.x) out[row * ld_out + c0 + i] = from_f<T>(sm[i] * inv * weight[c0 + i]);
+}
+
+}  // namespace dec
+}  // namespace gptb200

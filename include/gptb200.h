@@ -334,6 +334,42 @@ int gptb200_model_save_state(gptb200_model *m, const char *path);
 int gptb200_model_load_state(gptb200_model *m, const char *path);
 int gptb200_model_step_count(gptb200_model *m);
 
+/* ---- decoder models described by a folder with config.json and model.safetensors (no counterpart in the reference, whose one
+ *      model is GPT-2).  config.json names the architecture ("Budurax": Mamba-2 and latent-attention layers in any order, gated
+ *      GELU feed-forwards, layer norms before and after each sublayer, token shift, per-layer token input, depth average) and gives
+ *      every size and constant; gptb200_decoder_load chooses the model class by it.
+ *   dtype           GPTB200_DTYPE_BF16: weights, activations and caches in bf16, products on the tensor cores (up to eight rows:
+ *                   streamed weights) with fp32 accumulation; residual stream, norms, softmax and recurrences in fp32.
+ *                   GPTB200_DTYPE_F32: everything in fp32 FMAs.
+ *   open / close    a sequence's state for up to max_len tokens, zeroed; slots are reused after close
+ *   step            the next counts[i] tokens of each of n open slots (tokens: all of them, one slot after the other, host memory);
+ *                   want: rows of the step whose logits are wanted, logits: host, [n_want x vocab].  Returns when they are there.
+ *   generate        `steps` tokens for each of n slots: first[i] is the token at slot i's next position (sampled from its
+ *                   last logits); out (host) [steps x n].  One row per slot and step, the step replayed from a CUDA graph, sampling on
+ *                   the device: temperature 0 takes the largest logit, otherwise a draw from softmax(logits / temperature).  The
+ *                   last sampled token is not run.
+ *   message         receives the reason when loading fails (capacity bytes); later errors: gptb200_last_error(context).
+ *   options         "pass_rows" (most rows of one pass of a step, default 4096) and those of gptb200_ctx_set_option */
+typedef enum gptb200_dtype { GPTB200_DTYPE_BF16 = 0, GPTB200_DTYPE_F32 = 1 } gptb200_dtype;
+typedef struct gptb200_decoder gptb200_decoder;
+int gptb200_decoder_check_config(const char *config_json, char *message, size_t capacity);   /* host only */
+int gptb200_decoder_load(gptb200_decoder **out, const char *folder, int dtype, int device, void *cuda_stream, char *message, size_t capacity);
+int gptb200_decoder_destroy(gptb200_decoder *d);
+gptb200_ctx *gptb200_decoder_context(gptb200_decoder *d);
+int gptb200_decoder_vocab(gptb200_decoder *d);
+int gptb200_decoder_open(gptb200_decoder *d, int max_len, int *slot);
+int gptb200_decoder_close(gptb200_decoder *d, int slot);
+int gptb200_decoder_length(gptb200_decoder *d, int slot);   /* tokens the slot holds, -1: not open */
+int gptb200_decoder_set_option(gptb200_decoder *d, const char *key, int value);
+int gptb200_decoder_step(gptb200_decoder *d, int n, const int *slots, const int *counts, const int *tokens, int n_want, const int *want, float *logits);
+int gptb200_decoder_generate(gptb200_decoder *d, int n, const int *slots, const int *first, int steps, float temperature, unsigned long long seed, int *out);
+/* Frequencies of the dims / 2 rotated pairs and the factor on cosine and sine; scaling4 = {factor, original, fast, slow} (YaRN)
+ * or NULL.  Host only. */
+int gptb200_rotary_frequencies(int dims, double base, const double *scaling4, double *freq, double *gain);
+/* One token per row of logits (device, [rows x pitch]) into tokens (device): see generate.  draw: number of this call's draw. */
+int gptb200_sample_rows(gptb200_ctx *ctx, int *tokens, const float *logits, int rows, int vocab, long long pitch, float temperature, unsigned long long seed,
+                        unsigned long long draw);
+
 /* ---- token loader for data-parallel training: the reference's DataLoader (src/train/data_loader.h, data_loader.cpp:57-160)
  *      with the batch sharded over ranks.  Same file format (flat uint16 token ids) and the same sampling from the C
  *      library's rand() (seed it with srand, as src/train/train.cpp:73 does, identically on every rank): with world = 1 the
