@@ -42,7 +42,7 @@ EXPORTED_SYMBOLS = [
     "gptb200_bias_grad_noalloc",
     "gptb200_decoder_check_config", "gptb200_decoder_load", "gptb200_decoder_destroy", "gptb200_decoder_context", "gptb200_decoder_vocab",
     "gptb200_decoder_open", "gptb200_decoder_close", "gptb200_decoder_length", "gptb200_decoder_set_option", "gptb200_decoder_step",
-    "gptb200_decoder_generate", "gptb200_rotary_frequencies", "gptb200_sample_rows",
+    "gptb200_decoder_generate", "gptb200_rotary_frequencies", "gptb200_sample_rows", "gptb200_linear_bf16",
 ]
 
 

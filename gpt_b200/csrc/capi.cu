@@ -832,6 +832,11 @@ int run_gemm_batched(gptb200_ctx *ctx, float *out, long long out_ld, long long o
 
 int run_linear_bf16(gptb200_ctx *ctx, const Bf16Linear &c) { return run_linear_bf16_impl(ctx, c); }
 
+int bf16_operand_map(gptb200_ctx *ctx, CUtensorMap *map, const void *base, long long rows, long long cols, long long pitch, int box_rows)
+{
+    return make_word_tmap(ctx, map, base, rows, cols / 2, pitch / 2, kBK, box_rows, false);
+}
+
 int run_linear_f32(gptb200_ctx *ctx, float *out, const float *a, const float *w, int M, int N, int K)
 {
     GemmCall c{M, N, K, a, false, w, false, out, nullptr, nullptr, false};
@@ -1023,6 +1028,11 @@ int gptb200_ctx_set_option(gptb200_ctx *ctx, const char *key, int value)
     }
     if (!strcmp(key, "skinny_rowwise")) {
         ctx->skinny_rowwise = value != 0;
+        return GPTB200_OK;
+    }
+    if (!strcmp(key, "gemv_rows")) {
+        if (value < 0 || value > 8) return fail(ctx, GPTB200_ERR_INVALID_ARG, "gemv_rows must be 0 .. 8");
+        ctx->gemv_rows = value;
         return GPTB200_OK;
     }
     if (!strcmp(key, "decode_early_launch")) {
@@ -1297,6 +1307,20 @@ int gptb200_memcpy_d2h(gptb200_ctx *ctx, void *dst, const void *src, size_t byte
     CUDA_TRY(ctx, cudaMemcpyAsync(dst, src, bytes, cudaMemcpyDeviceToHost, ctx->stream));
     CUDA_TRY(ctx, cudaStreamSynchronize(ctx->stream));
     return GPTB200_OK;
+}
+
+int gptb200_linear_bf16(gptb200_ctx *ctx, int kind, void *out, long long out_pitch, const void *x, long long x_pitch, const void *w, int m, int n, int k, float *tail,
+                        int tail_col, int tail_pitch, const void *factor, const int *factor_rows, int factor_pitch)
+{
+    if (!ctx || kind < OUT_F32 || kind > OUT_GELU_MUL || m < 0 || n < 0 || k < 0) return GPTB200_ERR_INVALID_ARG;
+    if (m == 0 || n == 0) return GPTB200_OK;
+    if (!out || !x || !w || (kind == OUT_BF16 && tail_col < n && !tail) || (kind == OUT_GELU_MUL && (!factor || !factor_rows)))
+        return fail(ctx, GPTB200_ERR_INVALID_ARG, "null tensor pointer");
+    Bf16Linear c{};
+    c.M = m; c.N = n; c.K = k; c.a = x; c.lda = x_pitch; c.w = w; c.out_kind = kind; c.out = out; c.ldo = out_pitch;
+    c.tail = tail; c.tail_col = kind == OUT_BF16 ? tail_col : 0x7fffffff; c.tail_pitch = tail_pitch;
+    c.factor = factor; c.factor_rows = factor_rows; c.factor_pitch = factor_pitch;
+    return run_linear_bf16(ctx, c);
 }
 
 }  // extern "C"

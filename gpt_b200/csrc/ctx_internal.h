@@ -141,6 +141,10 @@ struct Bf16Linear {
 };
 int run_linear_bf16(gptb200_ctx *ctx, const Bf16Linear &c);
 
+// Tensor map of a bf16 matrix [rows][cols] with a row pitch (both in elements, multiples of 8): boxes of 64 columns x box_rows, 128-byte swizzle,
+// coordinates in 4-byte words (kept in the context like all maps).
+int bf16_operand_map(gptb200_ctx *ctx, CUtensorMap *map, const void *base, long long rows, long long cols, long long pitch, int box_rows);
+
 // out[m][n] = a[m][k] . w[n][k] in fp32 FMAs only (no tensor core), whatever the context's mode.
 int run_linear_f32(gptb200_ctx *ctx, float *out, const float *a, const float *w, int M, int N, int K);
 

@@ -19,6 +19,7 @@
 #include "decoder_config.h"
 #include "decoder_rows.cuh"
 #include "latent_attention.cuh"
+#include "latent_prefill_sm100.cuh"
 #include "mamba2.cuh"
 #include "safetensors.h"
 
@@ -70,6 +71,7 @@ public:
             if (s.base) cudaFree(s.base);
         for (void *p : weights_) cudaFree(p);
         for (void *p : work_) cudaFree(p);
+        if (expanded_) cudaFree(expanded_);
         if (host_) cudaFreeHost(host_);
     }
 
@@ -117,20 +119,27 @@ public:
             } else {
                 const LatentConfig &a = l.latent;
                 LatentShape &s = d.latent;
-                s = {a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, pad_to(a.kv_rank, 8), pad_to(a.kv_rank, 8) + pad_to(a.rot_dim, 8), a.rot.dims / 2, 0, 0,
-                     static_cast<float>(a.scale), 0, 0};
+                s = {a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, pad_to(a.kv_rank, 8), pad_to(a.kv_rank, 8) + pad_to(a.rot_dim, 16), pad_to(a.dim, 16), pad_to(a.vdim, 16),
+                     pad_to(a.dim, 16) + pad_to(a.rot_dim, 16), a.rot.dims / 2, 0, 0, static_cast<float>(a.scale), 0, 0};
                 d.own_keys = a.kv_from < 0;
                 const int nq = a.heads * (a.dim + a.rot_dim), nd = d.own_keys ? a.kv_rank + a.rot_dim : 0, ng = a.heads * a.vdim;
-                s.off_dkv = nq;
-                s.off_g = nq + nd;
-                d.proj_n = d.proj_cols = pad_to(nq + nd + ng, 8);
+                s.off_dkv = a.heads * s.q_stride;
+                s.off_g = s.off_dkv + pad_to(nd, 8);
+                d.proj_n = d.proj_cols = pad_to(s.off_g + ng, 8);
                 std::vector<Piece> pieces = {{m + "q", nq}};
                 if (d.own_keys) pieces.push_back({m + "dkv", nd});
                 pieces.push_back({m + "g", ng});
-                RC_TRY(matrix(file, &d.w_in, pieces, W, d.proj_n, pitch_));
+                const auto query_row = [&](int r) {
+                    const int h = r / (a.dim + a.rot_dim), i = r % (a.dim + a.rot_dim);
+                    return h * s.q_stride + (i < a.dim ? i : s.dim_pad + i - a.dim);
+                };
+                RC_TRY(matrix(file, &d.w_in, pieces, W, d.proj_n, pitch_, [&](int r) { return r < nq ? query_row(r) : r < nq + nd ? s.off_dkv + r - nq : s.off_g + r - nq - nd; }));
                 if (d.own_keys) RC_TRY(vector(file, &d.mix_norm, m + "dkv.norm", a.kv_rank));
-                RC_TRY(matrix(file, &d.w_uk, {{m + "uk", a.heads * a.dim}, {m + "uv", a.heads * a.vdim}}, a.kv_rank, a.heads * (a.dim + a.vdim), s.rank_pitch));
-                d.w_uv = d.w_uk + size_t(a.heads) * a.dim * s.rank_pitch;
+                RC_TRY(matrix(file, &d.w_uk, {{m + "uk", a.heads * a.dim}, {m + "uv", a.heads * a.vdim}}, a.kv_rank, a.heads * (s.dim_pad + s.v_pad), s.rank_pitch, [&](int r) {
+                    const int v = r - a.heads * a.dim;
+                    return v < 0 ? r / a.dim * s.dim_pad + r % a.dim : a.heads * s.dim_pad + v / a.vdim * s.v_pad + v % a.vdim;
+                }));
+                d.w_uv = d.w_uk + size_t(a.heads) * s.dim_pad * s.rank_pitch;
                 d.mix_out = pad_to(ng, 8);
                 RC_TRY(matrix(file, &d.w_o, {{m + "o", W}}, ng, pitch_, d.mix_out));
                 d.cache_owner = d.own_keys ? static_cast<int>(i) : a.kv_from;
@@ -230,6 +239,11 @@ public:
             pass_rows_ = value;
             return GPTB200_OK;
         }
+        if (!strcmp(key, "expand_rows")) {   // latent attention: shortest portion that takes the tensor-core form (0x7fffffff: none)
+            if (value < 1) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "expand_rows must be positive");
+            expand_rows_ = value;
+            return GPTB200_OK;
+        }
         return gptb200_ctx_set_option(ctx_, key, value);
     }
 
@@ -311,7 +325,7 @@ public:
         const GenerateControl control{seed, 0, temperature};
         CUDA_TRY(ctx_, cudaMemcpyAsync(gen_control_, &control, sizeof(control), cudaMemcpyHostToDevice, ctx_->stream));
         const auto body = [&]() -> int {
-            RC_TRY(kernels(n, n, n, longest));
+            RC_TRY(kernels(parts, n, n));
             RC_TRY(launch(sample_advance_kernel, dim3(n), dim3(512), 0, tokens_, history_, gen_control_, logits_, c_.vocab, vocab_pitch_, entries_));
             return launch(advance_step_kernel, dim3(1), dim3(1), 0, gen_control_);
         };
@@ -565,9 +579,7 @@ private:
         CUDA_TRY(ctx_, cudaStreamSynchronize(ctx_->stream));   // the pinned image and the logits of the previous pass are free
         RC_TRY(reserve(rows, static_cast<int>(want.size())));
         RC_TRY(upload(parts, tokens, rows, want));
-        int longest = 0;
-        for (const Part &p : parts) longest = std::max(longest, slots_[p.slot].length + p.count);
-        RC_TRY(kernels(static_cast<int>(parts.size()), rows, static_cast<int>(want.size()), longest));
+        RC_TRY(kernels(parts, rows, static_cast<int>(want.size())));
         for (const Part &p : parts) {
             slots_[p.slot].length += p.count;
             slots_[p.slot].parity ^= 1;
@@ -675,14 +687,84 @@ private:
     }
 
     template <int NR>
-    int latent_rows(const Layer &d, const LatentShape &s, int rows)
+    int latent_rows(const Layer &d, const LatentShape &s, int row0, int rows)
     {
         const size_t smem = (size_t(s.row_pitch) + size_t(kLatentWarps) * s.rank_pitch + 2 * kLatentWarps) * sizeof(float);
         return launch(latent_rows_kernel<T, NR>, dim3(s.heads, rows), dim3(kLatentWarps * 32), smem, act_, d.mix_out, static_cast<const T *>(proj_), static_cast<long long>(d.proj_cols),
-                      static_cast<const T *>(d.w_uk), static_cast<const T *>(d.w_uv), s, entries_, row_entry_);
+                      static_cast<const T *>(d.w_uk), static_cast<const T *>(d.w_uv), s, entries_, row_entry_, row0);
     }
 
-    int latent(const Layer &d, int n_entries, int rows, int longest)
+    int latent_absorbed(const Layer &d, int row0, int rows)
+    {
+        const LatentShape &s = d.latent;
+        if (s.row_pitch <= 128) return latent_rows<4>(d, s, row0, rows);
+        if (s.row_pitch <= 256) return latent_rows<8>(d, s, row0, rows);
+        if (s.row_pitch <= 384) return latent_rows<12>(d, s, row0, rows);
+        if (s.row_pitch <= 576) return latent_rows<18>(d, s, row0, rows);
+        return latent_rows<24>(d, s, row0, rows);
+    }
+
+    // Stages of the tensor-core kernel's rings; 0: its tiles do not fit (large heads), the absorbed form serves any number of rows.
+    int prefill_stages(const LatentShape &s, int *v_stages) const
+    {
+        const int u = (s.dim_pad + 63) / 64, r = (s.row_pitch - s.rank_pitch + 63) / 64, v = (s.v_pad + 63) / 64;
+        if (s.v_pad > 128) return 0;
+        for (const auto &st : {std::pair<int, int>{3, 3}, {2, 2}, {2, 1}, {1, 1}})
+            if (prefill_smem_bytes(u, r, v, st.first, st.second) <= 232448) {
+                *v_stages = st.second;
+                return st.first;
+            }
+        return 0;
+    }
+
+    // Expanded form for one request: keys and values of all its positions, then the tensor-core kernel.
+    int latent_expanded(const Layer &d, const Part &part)
+    {
+        if constexpr (kF32) {
+            return latent_absorbed(d, part.row0, part.count);
+        } else {
+            const LatentShape &s = d.latent;
+            const Slot &slot = slots_[part.slot];
+            const int positions = slot.length + part.count, cols = s.heads * (s.dim_pad + s.v_pad);
+            const size_t need = size_t(positions) * cols;
+            if (need > expanded_count_) {
+                CUDA_TRY(ctx_, cudaStreamSynchronize(ctx_->stream));
+                if (expanded_) CUDA_TRY(ctx_, cudaFree(expanded_));
+                expanded_ = nullptr;
+                expanded_count_ = 0;
+                void *p = nullptr;
+                CUDA_TRY(ctx_, cudaMalloc(&p, (need + need / 2) * sizeof(T)));
+                expanded_ = static_cast<T *>(p);
+                expanded_count_ = need + need / 2;
+            }
+            const T *cache = reinterpret_cast<const T *>(slot.base + s.cache_base + s.cache_per_position * slot.capacity);
+            Bf16Linear c{};
+            c.M = positions; c.N = cols; c.K = s.rank_pitch; c.a = cache; c.lda = s.row_pitch; c.w = d.w_uk; c.out_kind = OUT_BF16; c.out = expanded_; c.ldo = cols;
+            RC_TRY(run_linear_bf16(ctx_, c));
+            CUtensorMap mq, mkv, mc;
+            const T *q = proj_ + size_t(part.row0) * d.proj_cols;
+            RC_TRY(bf16_operand_map(ctx_, &mq, q, part.count, d.proj_cols, d.proj_cols, 128));
+            RC_TRY(bf16_operand_map(ctx_, &mkv, expanded_, positions, cols, cols, 128));
+            RC_TRY(bf16_operand_map(ctx_, &mc, cache, positions, s.row_pitch, s.row_pitch, 128));
+            PrefillParams p{};
+            p.rows = part.count; p.pos0 = slot.length;
+            p.heads = s.heads; p.vdim = s.vdim; p.v_pad = s.v_pad;
+            p.q_stride = s.q_stride; p.q_rot = s.dim_pad;
+            p.dim_pad = s.dim_pad; p.rot_pad = s.row_pitch - s.rank_pitch;
+            p.u_blocks = (p.dim_pad + 63) / 64; p.r_blocks = (p.rot_pad + 63) / 64; p.v_blocks = (s.v_pad + 63) / 64;
+            p.k_stages = prefill_stages(s, &p.v_stages);
+            p.v_col0 = s.heads * s.dim_pad;
+            p.rot_col0 = s.rank_pitch;
+            p.scale_log2 = static_cast<float>(static_cast<double>(s.scale) * 1.4426950408889634);
+            p.out = act_ + size_t(part.row0) * d.mix_out; p.ld_out = d.mix_out;
+            p.gate = q + s.off_g; p.ld_gate = d.proj_cols;
+            p.status = ctx_->d_status;
+            return launch(latent_prefill_kernel, dim3((part.count + 255) / 256, s.heads), dim3(kPrefillThreads),
+                          size_t(prefill_smem_bytes(p.u_blocks, p.r_blocks, p.v_blocks, p.k_stages, p.v_stages)), mq, mkv, mc, p);
+        }
+    }
+
+    int latent(const Layer &d, const std::vector<Part> &parts, int rows)
     {
         if constexpr (kF32) {
             RC_TRY(run_linear_f32(ctx_, proj_, h_, d.w_in, rows, d.proj_n, pitch_));
@@ -695,18 +777,27 @@ private:
         const float2 *table = table_ + rotaries_[d.rotary].table;
         RC_TRY(launch(latent_prepare_kernel<T>, dim3(rows), dim3(128), 0, proj_, static_cast<long long>(d.proj_cols), table, static_cast<const float *>(d.mix_norm),
                       static_cast<float>(c_.eps), s, d.own_keys ? 1 : 0, entries_, row_entry_));
-        (void)n_entries;
-        (void)longest;
-        if (s.row_pitch <= 128) return latent_rows<4>(d, s, rows);
-        if (s.row_pitch <= 256) return latent_rows<8>(d, s, rows);
-        if (s.row_pitch <= 384) return latent_rows<12>(d, s, rows);
-        if (s.row_pitch <= 576) return latent_rows<18>(d, s, rows);
-        return latent_rows<24>(d, s, rows);
+        // long portions one by one in the expanded form, runs of short ones together in the absorbed form
+        int v_stages = 0;
+        const bool tensor = !kF32 && prefill_stages(s, &v_stages) > 0;
+        for (size_t i = 0; i < parts.size();) {
+            if (tensor && parts[i].count >= expand_rows_) {
+                RC_TRY(latent_expanded(d, parts[i]));
+                ++i;
+                continue;
+            }
+            size_t j = i + 1;
+            while (j < parts.size() && !(tensor && parts[j].count >= expand_rows_)) ++j;
+            RC_TRY(latent_absorbed(d, parts[i].row0, parts[j - 1].row0 + parts[j - 1].count - parts[i].row0));
+            i = j;
+        }
+        return GPTB200_OK;
     }
 
     // All kernels of one step; everything that changes from step to step is read from device memory.
-    int kernels(int n_entries, int rows, int n_want, int longest)
+    int kernels(const std::vector<Part> &parts, int rows, int n_want)
     {
+        const int n_entries = static_cast<int>(parts.size());
         const float eps = static_cast<float>(c_.eps);
         RC_TRY(launch(embed_rows_kernel<T>, dim3(rows), dim3(row_threads()), 0, states_, static_cast<const T *>(embed_), static_cast<const int *>(tokens_), pitch_));
         for (const Rotary &r : rotaries_)
@@ -716,7 +807,7 @@ private:
             const Layer &d = layers_[i];
             float *x = x_[i & 1];
             RC_TRY(layer_begin(rows, static_cast<int>(i), h_, nullptr));
-            RC_TRY(c_.layers[i].kind == MixerKind::Mamba2 ? mamba(d, n_entries, rows) : latent(d, n_entries, rows, longest));
+            RC_TRY(c_.layers[i].kind == MixerKind::Mamba2 ? mamba(d, n_entries, rows) : latent(d, parts, rows));
             RC_TRY(linear_f32(y_, act_, d.w_o, rows, pitch_, d.mix_out));
             const size_t smem = size_t(pitch_) * sizeof(float);
             RC_TRY(launch(sublayer_end_kernel<T>, dim3(rows), dim3(row_threads()), smem, x, static_cast<const float *>(y_), static_cast<const float *>(d.norm1b.w),
@@ -763,7 +854,9 @@ private:
     size_t fixed_state_ = 0, position_bytes_ = 0;
     std::vector<void *> weights_, work_;
     std::vector<Slot> slots_;
-    int pass_rows_ = 4096;
+    int pass_rows_ = 4096, expand_rows_ = 32;
+    T *expanded_ = nullptr;
+    size_t expanded_count_ = 0;
     int rows_ = 0, wanted_ = 0;
     long long state_stride_ = 0;
     float *states_ = nullptr, *x_[2] = {nullptr, nullptr}, *y_ = nullptr, *tail_ = nullptr, *dt_ = nullptr, *decay_ = nullptr, *ssm_y_ = nullptr, *glu_ = nullptr, *logits_ = nullptr;

@@ -1,7 +1,7 @@
 // Latent attention (multi-head attention whose keys and values are linear maps of one small latent per token).
 //
-// Only the normed latent c and the rotated key part shared by all heads are cached: a row per position, [c | rotated key] in T, each
-// part padded to a multiple of 8.  Two forms of the same attention:
+// Only the normed latent c and the rotated key part shared by all heads are cached: a row per position, [c | rotated key] in T, the
+// parts padded with zeros.  Two forms of the same attention:
 //   absorbed   scores against the cached rows themselves: q_u . (W_uk c) = (W_uk^T q_u) . c, and W_uv is applied to the weighted
 //              sum of latents (few rows: decoding, short portions; and all fp32 work)
 //   expanded   keys and values of all visible positions as matrices, tensor-core attention over them (prompts)
@@ -15,7 +15,9 @@ namespace dec {
 
 struct LatentShape {
     int heads, dim, rot_dim, vdim, kv_rank;
-    int rank_pitch, row_pitch;    // kv_rank padded; cached row [c | rotated key part]
+    int rank_pitch, row_pitch;    // kv_rank padded to 8; cached row [c | rotated key part padded to 16]
+    int dim_pad, v_pad;           // rows of W_uk / W_uv per head (dim and vdim padded to 16, zero rows)
+    int q_stride;                 // projection columns per head: [unrotated: dim_pad | rotated, padded to 16]
     int rot_half;                 // rotated pairs
     int off_dkv, off_g;           // columns of W_dkv h and W_g h in the projection row (q starts at 0)
     float scale;
@@ -59,7 +61,7 @@ __global__ void latent_prepare_kernel(T *__restrict__ proj, long long ld, const 
     const float2 *cs = table + static_cast<long long>(row) * s.rot_half;
     for (int i = threadIdx.x; i < s.heads * s.rot_half; i += blockDim.x) {
         const int h = i / s.rot_half, k = i % s.rot_half;
-        T *q = r + h * (s.dim + s.rot_dim) + s.dim + k;
+        T *q = r + h * s.q_stride + s.dim_pad + k;
         const float u = to_f(q[0]), v = to_f(q[s.rot_half]);
         q[0] = from_f<T>(u * cs[k].x - v * cs[k].y);
         q[s.rot_half] = from_f<T>(v * cs[k].x + u * cs[k].y);
@@ -92,11 +94,11 @@ constexpr int kLatentWarps = 4;
 
 // Absorbed form, one block per (head, row): the query is mapped into the latent space, every warp goes through every fourth
 // visible position with a running maximum and sum, the warps' parts are merged, W_uv and the output gate are applied.
-// NR: cached row values per lane.  w_uk [heads * dim][rank_pitch], w_uv [heads * vdim][rank_pitch].
+// NR: cached row values per lane.  w_uk [heads * dim_pad][rank_pitch], w_uv [heads * v_pad][rank_pitch].
 template <typename T, int NR>
 __global__ void __launch_bounds__(kLatentWarps * 32)
 latent_rows_kernel(T *__restrict__ out, int ld_out, const T *__restrict__ proj, long long ld, const T *__restrict__ w_uk, const T *__restrict__ w_uv,
-                   const LatentShape s, const StepEntry *__restrict__ entries, const int *__restrict__ row_entry)
+                   const LatentShape s, const StepEntry *__restrict__ entries, const int *__restrict__ row_entry, int row0)
 {
     extern __shared__ float sm[];
     float *q = sm;                                   // [row_pitch] query in the cached rows' space
@@ -104,18 +106,18 @@ latent_rows_kernel(T *__restrict__ out, int ld_out, const T *__restrict__ proj, 
     float *ml = acc_sm + kLatentWarps * s.rank_pitch;   // [warps][2]
     grid_dependency_wait();
     grid_dependency_launch();
-    const int h = blockIdx.x, row = blockIdx.y;
+    const int h = blockIdx.x, row = row0 + blockIdx.y;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const StepEntry e = entries[row_entry[row]];
     const int last = e.pos0 + row - e.row0;          // this row's position
-    const T *qr = proj + row * ld + h * (s.dim + s.rot_dim);
+    const T *qr = proj + row * ld + h * s.q_stride;
     for (int j = threadIdx.x; j < s.row_pitch; j += blockDim.x) {
         float v = 0.0f;
         if (j < s.kv_rank) {
-            const T *w = w_uk + static_cast<long long>(h) * s.dim * s.rank_pitch + j;
+            const T *w = w_uk + static_cast<long long>(h) * s.dim_pad * s.rank_pitch + j;
             for (int d = 0; d < s.dim; ++d) v = fmaf(to_f(qr[d]), to_f(w[static_cast<long long>(d) * s.rank_pitch]), v);
         } else if (j >= s.rank_pitch && j - s.rank_pitch < s.rot_dim) {
-            v = to_f(qr[s.dim + j - s.rank_pitch]);
+            v = to_f(qr[s.dim_pad + j - s.rank_pitch]);
         }
         q[j] = v * s.scale;
     }
@@ -168,7 +170,7 @@ latent_rows_kernel(T *__restrict__ out, int ld_out, const T *__restrict__ proj, 
     }
     __syncthreads();
     for (int n = warp; n < s.vdim; n += kLatentWarps) {
-        const T *w = w_uv + (static_cast<long long>(h) * s.vdim + n) * s.rank_pitch;
+        const T *w = w_uv + (static_cast<long long>(h) * s.v_pad + n) * s.rank_pitch;
         float v = 0.0f;
         for (int j = lane; j < s.kv_rank; j += 32) v = fmaf(to_f(w[j]), q[j], v);
 #pragma unroll

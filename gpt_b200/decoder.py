@@ -37,6 +37,7 @@ def load_library() -> ctypes.CDLL:
         "gptb200_decoder_step": (i, [vp, i, vp, vp, vp, i, vp, vp]),
         "gptb200_decoder_generate": (i, [vp, i, vp, vp, i, f32, ull, vp]),
         "gptb200_rotary_frequencies": (i, [i, ctypes.c_double, dp, dp, dp]),
+        "gptb200_linear_bf16": (i, [vp, i, vp, ll, vp, ll, vp, i, i, i, vp, i, i, vp, vp, i]),
         "gptb200_sample_rows": (i, [vp, vp, vp, i, i, ll, f32, ull, ull]),
         "gptb200_ctx_launch_count": (ll, [vp]),
         "gptb200_ctx_synchronize": (i, [vp]),

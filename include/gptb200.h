@@ -83,6 +83,7 @@ int gptb200_ctx_set_stream(gptb200_ctx *ctx, void *cuda_stream);
  * time, because the kernel runs at the board's power limit and the clock drops by as much; one more launch per GEMM),
  * "fuse_dbias" (weight-gradient launches of the CTA-pair kernel also produce the bias gradient: 1 = on (default), 0 = the
  * separate column-sum kernels; results differ only in summation order),
+ * "gemv_rows" (gptb200_linear_bf16: most rows the weight-streaming kernel takes, 0 .. 8, default 8),
  * "max_sms" (0 = all SMs; otherwise the GEMM kernels occupy at most this many, which leaves SMs to a collective that runs
  * at the same time on another stream),
  * "trace" (record a kernel-phase trace of each CTA-pair GEMM launch: 1 = on, 0 = off (default)),
@@ -349,7 +350,8 @@ int gptb200_model_step_count(gptb200_model *m);
  *                   the device: temperature 0 takes the largest logit, otherwise a draw from softmax(logits / temperature).  The
  *                   last sampled token is not run.
  *   message         receives the reason when loading fails (capacity bytes); later errors: gptb200_last_error(context).
- *   options         "pass_rows" (most rows of one pass of a step, default 4096) and those of gptb200_ctx_set_option */
+ *   options         "pass_rows" (most rows of one pass of a step, default 4096), "expand_rows" (latent attention in bf16: shortest portion
+ *                   whose keys and values are expanded for the tensor cores, default 32; shorter ones use the latents as they are) and those of gptb200_ctx_set_option */
 typedef enum gptb200_dtype { GPTB200_DTYPE_BF16 = 0, GPTB200_DTYPE_F32 = 1 } gptb200_dtype;
 typedef struct gptb200_decoder gptb200_decoder;
 int gptb200_decoder_check_config(const char *config_json, char *message, size_t capacity);   /* host only */
@@ -366,6 +368,15 @@ int gptb200_decoder_generate(gptb200_decoder *d, int n, const int *slots, const 
 /* Frequencies of the dims / 2 rotated pairs and the factor on cosine and sine; scaling4 = {factor, original, fast, slow} (YaRN)
  * or NULL.  Host only. */
 int gptb200_rotary_frequencies(int dims, double base, const double *scaling4, double *freq, double *gain);
+/* out[m x n] = x[m x k] . w[n x k]^T with bf16 operands and fp32 accumulation: the product behind every linear layer of these
+ * models.  w is contiguous; pitches are in elements; k and the pitches are multiples of 8, addresses 16-byte aligned.
+ *   kind 0  out fp32
+ *        1  out bf16; columns from tail_col (a multiple of 32; n or more: none) on stay fp32 and go to tail [m x tail_pitch]
+ *        2  gated: columns of w come in groups of 32 gate | 32 up (n a multiple of 64), out bf16 [m x n/2] = gelu_tanh(gate) * up
+ *        3  out bf16 = gelu_tanh(product) * factor[factor_rows[row]][column], factor bf16 with row pitch factor_pitch (n a multiple of 8)
+ * Up to 8 rows (option "gemv_rows") a weight-streaming kernel, else the tcgen05 kernels. */
+int gptb200_linear_bf16(gptb200_ctx *ctx, int kind, void *out, long long out_pitch, const void *x, long long x_pitch, const void *w, int m, int n, int k, float *tail,
+                        int tail_col, int tail_pitch, const void *factor, const int *factor_rows, int factor_pitch);
 /* One token per row of logits (device, [rows x pitch]) into tokens (device): see generate.  draw: number of this call's draw. */
 int gptb200_sample_rows(gptb200_ctx *ctx, int *tokens, const float *logits, int rows, int vocab, long long pitch, float temperature, unsigned long long seed,
                         unsigned long long draw);
