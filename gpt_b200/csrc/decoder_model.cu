@@ -21,6 +21,7 @@
 #include "latent_attention.cuh"
 #include "latent_prefill_sm100.cuh"
 #include "mamba2.cuh"
+#include "mamba2_chunk.cuh"
 #include "safetensors.h"
 
 using namespace gptb200;
@@ -237,6 +238,11 @@ public:
         if (!strcmp(key, "pass_rows")) {   // most rows of one pass: longer steps are worked through in several
             if (value < 1) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "pass_rows must be positive");
             pass_rows_ = value;
+            return GPTB200_OK;
+        }
+        if (!strcmp(key, "chunk_rows")) {   // Mamba-2: shortest portion that takes the chunked tensor-core form (0x7fffffff: none)
+            if (value < 1) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "chunk_rows must be positive");
+            chunk_rows_ = value;
             return GPTB200_OK;
         }
         if (!strcmp(key, "expand_rows")) {   // latent attention: shortest portion that takes the tensor-core form (0x7fffffff: none)
@@ -654,7 +660,7 @@ private:
         return launch(layer_begin_kernel<T>, dim3((rows + b.tile - 1) / b.tile), dim3(row_threads()), 2 * size_t(pitch_) * sizeof(float), b);
     }
 
-    int mamba(const Layer &d, int n_entries, int rows)
+    int mamba(const Layer &d, const std::vector<Part> &parts, int rows)
     {
         const MambaShape &s = d.mamba;
         const float *dt_raw = tail_;
@@ -675,15 +681,38 @@ private:
         RC_TRY(launch(mamba_conv_kernel<T>, dim3(conv_blocks + dt_blocks, rows), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, static_cast<const T *>(proj_), ld, dt_raw, ld_dt,
                       static_cast<const float *>(d.taps), static_cast<const float *>(d.conv_b), static_cast<const float *>(d.dt_bias), static_cast<const float *>(d.a_log), s, entries_,
                       row_entry_, conv_blocks));
+        // long portions in chunks on the tensor cores, short ones token by token; neighbours of a kind in one launch
+        const bool chunks = !kF32 && s.state <= kChunkMaxState;
+        for (size_t i = 0, j; i < parts.size(); i = j) {
+            const bool longer = chunks && parts[i].count >= chunk_rows_;
+            for (j = i + 1; j < parts.size() && (chunks && parts[j].count >= chunk_rows_) == longer;) ++j;
+            RC_TRY(longer ? mamba_chunks(d, static_cast<int>(i), static_cast<int>(j - i), ld_xbc) : mamba_tokens(d, static_cast<int>(i), static_cast<int>(j - i), ld_xbc));
+        }
+        const int part = s.inner / s.norm_groups;
+        return launch(mamba_gated_norm_kernel<T>, dim3(rows, s.norm_groups), dim3(std::min(256, pad_to(part, 32))), size_t(part) * sizeof(float), act_, d.mix_out,
+                      static_cast<const float *>(ssm_y_), static_cast<const T *>(proj_), ld, static_cast<const float *>(d.mix_norm), s, static_cast<float>(c_.eps));
+    }
+
+    int mamba_chunks(const Layer &d, int entry0, int n, int ld_xbc)
+    {
+        if constexpr (kF32) {
+            return mamba_tokens(d, entry0, n, ld_xbc);
+        } else {
+            const MambaShape &s = d.mamba;
+            return launch(mamba_chunk_kernel, dim3(s.heads * ((s.vdim + kChunkCols - 1) / kChunkCols), n), dim3(kChunkThreads), size_t(chunk_smem_bytes(s.state)), ssm_y_, xbc_, ld_xbc, dt_,
+                          decay_, d.d_skip, s, entries_ + entry0);
+        }
+    }
+
+    int mamba_tokens(const Layer &d, int entry0, int n, int ld_xbc)
+    {
+        const MambaShape &s = d.mamba;
         const int threads = std::max(256, pad_to(s.vdim, 32));
         if (threads > 1024) return fail(ctx_, GPTB200_ERR_TOO_LARGE, "mamba2: vdim beyond 1024");
         const size_t smem = (size_t(s.state) * s.vdim + size_t(threads / s.vdim) * s.vdim + 2 * s.state + s.vdim) * sizeof(float);
         if (smem > 227 * 1024) return fail(ctx_, GPTB200_ERR_TOO_LARGE, "mamba2: a head's state does not fit in shared memory");
-        RC_TRY(launch(mamba_scan_kernel<T>, dim3(s.heads, n_entries), dim3(threads), smem, ssm_y_, static_cast<const T *>(xbc_), ld_xbc, static_cast<const float *>(dt_),
-                      static_cast<const float *>(decay_), static_cast<const float *>(d.d_skip), s, entries_));
-        const int part = s.inner / s.norm_groups;
-        return launch(mamba_gated_norm_kernel<T>, dim3(rows, s.norm_groups), dim3(std::min(256, pad_to(part, 32))), size_t(part) * sizeof(float), act_, d.mix_out,
-                      static_cast<const float *>(ssm_y_), static_cast<const T *>(proj_), ld, static_cast<const float *>(d.mix_norm), s, static_cast<float>(c_.eps));
+        return launch(mamba_scan_kernel<T>, dim3(s.heads, n), dim3(threads), smem, ssm_y_, static_cast<const T *>(xbc_), ld_xbc, static_cast<const float *>(dt_),
+                      static_cast<const float *>(decay_), static_cast<const float *>(d.d_skip), s, entries_ + entry0);
     }
 
     template <int NR>
@@ -797,7 +826,6 @@ private:
     // All kernels of one step; everything that changes from step to step is read from device memory.
     int kernels(const std::vector<Part> &parts, int rows, int n_want)
     {
-        const int n_entries = static_cast<int>(parts.size());
         const float eps = static_cast<float>(c_.eps);
         RC_TRY(launch(embed_rows_kernel<T>, dim3(rows), dim3(row_threads()), 0, states_, static_cast<const T *>(embed_), static_cast<const int *>(tokens_), pitch_));
         for (const Rotary &r : rotaries_)
@@ -807,7 +835,7 @@ private:
             const Layer &d = layers_[i];
             float *x = x_[i & 1];
             RC_TRY(layer_begin(rows, static_cast<int>(i), h_, nullptr));
-            RC_TRY(c_.layers[i].kind == MixerKind::Mamba2 ? mamba(d, n_entries, rows) : latent(d, parts, rows));
+            RC_TRY(c_.layers[i].kind == MixerKind::Mamba2 ? mamba(d, parts, rows) : latent(d, parts, rows));
             RC_TRY(linear_f32(y_, act_, d.w_o, rows, pitch_, d.mix_out));
             const size_t smem = size_t(pitch_) * sizeof(float);
             RC_TRY(launch(sublayer_end_kernel<T>, dim3(rows), dim3(row_threads()), smem, x, static_cast<const float *>(y_), static_cast<const float *>(d.norm1b.w),
@@ -854,7 +882,7 @@ private:
     size_t fixed_state_ = 0, position_bytes_ = 0;
     std::vector<void *> weights_, work_;
     std::vector<Slot> slots_;
-    int pass_rows_ = 4096, expand_rows_ = 32;
+    int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8;
     T *expanded_ = nullptr;
     size_t expanded_count_ = 0;
     int rows_ = 0, wanted_ = 0;
