@@ -19,6 +19,7 @@
 #include "decoder_config.h"
 #include "decoder_rows.cuh"
 #include "latent_attention.cuh"
+#include "latent_decode.cuh"
 #include "latent_prefill_sm100.cuh"
 #include "mamba2.cuh"
 #include "mamba2_chunk.cuh"
@@ -73,6 +74,7 @@ public:
         for (void *p : weights_) cudaFree(p);
         for (void *p : work_) cudaFree(p);
         if (expanded_) cudaFree(expanded_);
+        if (scratch_) cudaFree(scratch_);
         if (host_) cudaFreeHost(host_);
     }
 
@@ -120,7 +122,7 @@ public:
             } else {
                 const LatentConfig &a = l.latent;
                 LatentShape &s = d.latent;
-                s = {a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, pad_to(a.kv_rank, 8), pad_to(a.kv_rank, 8) + pad_to(a.rot_dim, 16), pad_to(a.dim, 16), pad_to(a.vdim, 16),
+                s = {a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, pad_to(a.kv_rank, 16), pad_to(a.kv_rank, 16) + pad_to(a.rot_dim, 16), pad_to(a.dim, 16), pad_to(a.vdim, 16),
                      pad_to(a.dim, 16) + pad_to(a.rot_dim, 16), a.rot.dims / 2, 0, 0, static_cast<float>(a.scale), 0, 0};
                 d.own_keys = a.kv_from < 0;
                 const int nq = a.heads * (a.dim + a.rot_dim), nd = d.own_keys ? a.kv_rank + a.rot_dim : 0, ng = a.heads * a.vdim;
@@ -146,6 +148,7 @@ public:
                 d.cache_owner = d.own_keys ? static_cast<int>(i) : a.kv_from;
                 d.rotary = rotary_index(a.rot);
                 if (s.row_pitch > 768) return fail(ctx_, GPTB200_ERR_TOO_LARGE, "latent attention: kv_rank + rot_dim beyond 768");
+                if (a.dim > 1024) return fail(ctx_, GPTB200_ERR_TOO_LARGE, "latent attention: dim beyond 1024");
             }
             if (l.ff > 0) {
                 RC_TRY(norm(file, &d.norm2, p + "norm2"));
@@ -331,7 +334,10 @@ public:
         const GenerateControl control{seed, 0, temperature};
         CUDA_TRY(ctx_, cudaMemcpyAsync(gen_control_, &control, sizeof(control), cudaMemcpyHostToDevice, ctx_->stream));
         const auto body = [&]() -> int {
-            RC_TRY(kernels(parts, n, n));
+            generating_ = true;
+            const int rc = kernels(parts, n, n);
+            generating_ = false;
+            RC_TRY(rc);
             RC_TRY(launch(sample_advance_kernel, dim3(n), dim3(512), 0, tokens_, history_, gen_control_, logits_, c_.vocab, vocab_pitch_, entries_));
             return launch(advance_step_kernel, dim3(1), dim3(1), 0, gen_control_);
         };
@@ -676,17 +682,22 @@ private:
             c.tail = tail_; c.tail_col = d.proj_cols; c.tail_pitch = ld_dt;
             RC_TRY(run_linear_bf16(ctx_, c));
         }
-        const int ld_xbc = pad_to(s.channels, 8);
-        const int conv_blocks = (s.channels + 127) / 128, dt_blocks = (s.heads + 127) / 128;
-        RC_TRY(launch(mamba_conv_kernel<T>, dim3(conv_blocks + dt_blocks, rows), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, static_cast<const T *>(proj_), ld, dt_raw, ld_dt,
-                      static_cast<const float *>(d.taps), static_cast<const float *>(d.conv_b), static_cast<const float *>(d.dt_bias), static_cast<const float *>(d.a_log), s, entries_,
-                      row_entry_, conv_blocks));
-        // long portions in chunks on the tensor cores, short ones token by token; neighbours of a kind in one launch
-        const bool chunks = !kF32 && s.state <= kChunkMaxState;
+        // single tokens in one launch; long portions in chunks on the tensor cores, short ones token by token, both behind the
+        // convolution kernel; neighbours of a kind together
+        const auto kind = [&](const Part &p) { return p.count == 1 ? 0 : !kF32 && s.state <= kChunkMaxState && p.count >= chunk_rows_ ? 2 : 1; };
         for (size_t i = 0, j; i < parts.size(); i = j) {
-            const bool longer = chunks && parts[i].count >= chunk_rows_;
-            for (j = i + 1; j < parts.size() && (chunks && parts[j].count >= chunk_rows_) == longer;) ++j;
-            RC_TRY(longer ? mamba_chunks(d, static_cast<int>(i), static_cast<int>(j - i), ld_xbc) : mamba_tokens(d, static_cast<int>(i), static_cast<int>(j - i), ld_xbc));
+            const int k = kind(parts[i]);
+            for (j = i + 1; j < parts.size() && kind(parts[j]) == k;) ++j;
+            const int entry0 = static_cast<int>(i), n = static_cast<int>(j - i), row0 = parts[i].row0, run = parts[j - 1].row0 + parts[j - 1].count - row0;
+            if (k == 0) {
+                RC_TRY(launch(mamba_step_kernel<T>, dim3(s.heads * ((s.vdim + kStepCols - 1) / kStepCols), n), dim3(256), (2 * size_t(s.state) + 9 * kStepCols) * sizeof(float), ssm_y_, proj_, ld,
+                              dt_raw, ld_dt, d.taps, d.conv_b, d.dt_bias, d.a_log, d.d_skip, s, entries_ + entry0));
+                continue;
+            }
+            const int ld_xbc = pad_to(s.channels, 8), conv_blocks = (s.channels + 127) / 128, dt_blocks = (s.heads + 127) / 128;
+            RC_TRY(launch(mamba_conv_kernel<T>, dim3(conv_blocks + dt_blocks, run), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, proj_, ld, dt_raw, ld_dt, d.taps, d.conv_b, d.dt_bias, d.a_log, s,
+                          entries_, row_entry_, conv_blocks, row0));
+            RC_TRY(k == 2 ? mamba_chunks(d, entry0, n, ld_xbc) : mamba_tokens(d, entry0, n, ld_xbc));
         }
         const int part = s.inner / s.norm_groups;
         return launch(mamba_gated_norm_kernel<T>, dim3(rows, s.norm_groups), dim3(std::min(256, pad_to(part, 32))), size_t(part) * sizeof(float), act_, d.mix_out,
@@ -723,14 +734,49 @@ private:
                       static_cast<const T *>(d.w_uk), static_cast<const T *>(d.w_uv), s, entries_, row_entry_, row0);
     }
 
-    int latent_absorbed(const Layer &d, int row0, int rows)
+    // positions: most that any of the rows sees (an upper bound)
+    int latent_absorbed(const Layer &d, int row0, int rows, int positions)
     {
         const LatentShape &s = d.latent;
-        if (s.row_pitch <= 128) return latent_rows<4>(d, s, row0, rows);
-        if (s.row_pitch <= 256) return latent_rows<8>(d, s, row0, rows);
-        if (s.row_pitch <= 384) return latent_rows<12>(d, s, row0, rows);
-        if (s.row_pitch <= 576) return latent_rows<18>(d, s, row0, rows);
-        return latent_rows<24>(d, s, row0, rows);
+        if constexpr (kF32) {
+            (void)positions;
+            RC_TRY(latent_prepare(d, row0, rows));
+            if (s.row_pitch <= 128) return latent_rows<4>(d, s, row0, rows);
+            if (s.row_pitch <= 256) return latent_rows<8>(d, s, row0, rows);
+            if (s.row_pitch <= 384) return latent_rows<12>(d, s, row0, rows);
+            if (s.row_pitch <= 576) return latent_rows<18>(d, s, row0, rows);
+            return latent_rows<24>(d, s, row0, rows);
+        } else {
+            // ranges of positions: enough blocks for the machine, at least two tiles each
+            const int groups = (s.heads + 15) / 16;
+            int splits = std::max(1, 2 * ctx_->num_sms / (rows * groups));
+            splits = std::min({splits, 128, std::max(1, (positions + 2 * kSplitTile - 1) / (2 * kSplitTile))});
+            const size_t q_count = size_t(rows) * s.heads * s.row_pitch, o_count = size_t(rows) * s.heads * splits * s.rank_pitch, ml_count = size_t(rows) * s.heads * splits * 2;
+            RC_TRY(scratch(q_count + o_count + ml_count));
+            float *q = scratch_, *o = q + q_count, *ml = o + o_count;
+            const int slices = (s.rank_pitch + kQuerySlice - 1) / kQuerySlice;
+            RC_TRY(launch(latent_query_kernel, dim3(s.heads * slices + (d.own_keys ? 1 : 0), rows), dim3(256), 0, q, proj_, d.proj_cols, d.w_uk, table_ + rotaries_[d.rotary].table,
+                          d.mix_norm, static_cast<float>(c_.eps), s, entries_, row_entry_, row0));
+            RC_TRY(launch(latent_split_kernel, dim3(splits, groups, rows), dim3(kSplitThreads), size_t(split_smem_bytes(s.row_pitch)), o, ml, q, s, entries_, row_entry_, row0));
+            return launch(latent_combine_kernel, dim3(s.heads * ((s.vdim + kCombineRows - 1) / kCombineRows), rows), dim3(256), size_t(s.rank_pitch) * sizeof(float), act_, d.mix_out, o, ml,
+                          splits, proj_, d.proj_cols, d.w_uv, s, entries_, row_entry_, row0);
+        }
+    }
+
+    // fp32 scratch of the absorbed form (grown on demand; a captured step keeps its address)
+    int scratch(size_t count)
+    {
+        if (count <= scratch_count_) return GPTB200_OK;
+        CUDA_TRY(ctx_, cudaStreamSynchronize(ctx_->stream));
+        drop_graph();
+        if (scratch_) CUDA_TRY(ctx_, cudaFree(scratch_));
+        scratch_ = nullptr;
+        scratch_count_ = 0;
+        void *p = nullptr;
+        CUDA_TRY(ctx_, cudaMalloc(&p, count * sizeof(float)));
+        scratch_ = static_cast<float *>(p);
+        scratch_count_ = count;
+        return GPTB200_OK;
     }
 
     // Stages of the tensor-core kernel's rings; 0: its tiles do not fit (large heads), the absorbed form serves any number of rows.
@@ -750,7 +796,7 @@ private:
     int latent_expanded(const Layer &d, const Part &part)
     {
         if constexpr (kF32) {
-            return latent_absorbed(d, part.row0, part.count);
+            return latent_absorbed(d, part.row0, part.count, 0);
         } else {
             const LatentShape &s = d.latent;
             const Slot &slot = slots_[part.slot];
@@ -803,24 +849,32 @@ private:
             RC_TRY(run_linear_bf16(ctx_, c));
         }
         const LatentShape &s = d.latent;
-        const float2 *table = table_ + rotaries_[d.rotary].table;
-        RC_TRY(launch(latent_prepare_kernel<T>, dim3(rows), dim3(128), 0, proj_, static_cast<long long>(d.proj_cols), table, static_cast<const float *>(d.mix_norm),
-                      static_cast<float>(c_.eps), s, d.own_keys ? 1 : 0, entries_, row_entry_));
         // long portions one by one in the expanded form, runs of short ones together in the absorbed form
         int v_stages = 0;
         const bool tensor = !kF32 && prefill_stages(s, &v_stages) > 0;
         for (size_t i = 0; i < parts.size();) {
             if (tensor && parts[i].count >= expand_rows_) {
+                RC_TRY(latent_prepare(d, parts[i].row0, parts[i].count));
                 RC_TRY(latent_expanded(d, parts[i]));
                 ++i;
                 continue;
             }
-            size_t j = i + 1;
-            while (j < parts.size() && !(tensor && parts[j].count >= expand_rows_)) ++j;
-            RC_TRY(latent_absorbed(d, parts[i].row0, parts[j - 1].row0 + parts[j - 1].count - parts[i].row0));
+            size_t j = i;
+            int positions = 0;
+            for (; j < parts.size() && !(tensor && parts[j].count >= expand_rows_); ++j) {
+                const Slot &slot = slots_[parts[j].slot];
+                positions = std::max(positions, generating_ ? slot.capacity : slot.length + parts[j].count);
+            }
+            RC_TRY(latent_absorbed(d, parts[i].row0, parts[j - 1].row0 + parts[j - 1].count - parts[i].row0, positions));
             i = j;
         }
         return GPTB200_OK;
+    }
+
+    int latent_prepare(const Layer &d, int row0, int rows)
+    {
+        return launch(latent_prepare_kernel<T>, dim3(rows), dim3(128), 0, proj_, d.proj_cols, table_ + rotaries_[d.rotary].table, d.mix_norm, static_cast<float>(c_.eps), d.latent,
+                      d.own_keys ? 1 : 0, entries_, row_entry_, row0);
     }
 
     // All kernels of one step; everything that changes from step to step is read from device memory.
@@ -885,6 +939,9 @@ private:
     int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8;
     T *expanded_ = nullptr;
     size_t expanded_count_ = 0;
+    float *scratch_ = nullptr;
+    size_t scratch_count_ = 0;
+    bool generating_ = false;   // launches must serve every length up to the slots' capacities
     int rows_ = 0, wanted_ = 0;
     long long state_stride_ = 0;
     float *states_ = nullptr, *x_[2] = {nullptr, nullptr}, *y_ = nullptr, *tail_ = nullptr, *dt_ = nullptr, *decay_ = nullptr, *ssm_y_ = nullptr, *glu_ = nullptr, *logits_ = nullptr;

@@ -15,7 +15,7 @@ namespace dec {
 
 struct LatentShape {
     int heads, dim, rot_dim, vdim, kv_rank;
-    int rank_pitch, row_pitch;    // kv_rank padded to 8; cached row [c | rotated key part padded to 16]
+    int rank_pitch, row_pitch;    // kv_rank padded to 16; cached row [c | rotated key part padded to 16]
     int dim_pad, v_pad;           // rows of W_uk / W_uv per head (dim and vdim padded to 16, zero rows)
     int q_stride;                 // projection columns per head: [unrotated: dim_pad | rotated, padded to 16]
     int rot_half;                 // rotated pairs
@@ -46,16 +46,25 @@ __global__ void rotary_table_kernel(float2 *__restrict__ table, const double *__
     table[i] = make_float2(static_cast<float>(c * gain), static_cast<float>(s * gain));
 }
 
+// Component k of a rotated part x (rotated pairs, then dimensions that pass unchanged, then zeros for the padding).
+template <typename T>
+__device__ __forceinline__ float rotated(const T *x, int k, const float2 *cs, const LatentShape &s)
+{
+    if (k < s.rot_half) return to_f(x[k]) * cs[k].x - to_f(x[k + s.rot_half]) * cs[k].y;
+    if (k < 2 * s.rot_half) return to_f(x[k]) * cs[k - s.rot_half].x + to_f(x[k - s.rot_half]) * cs[k - s.rot_half].y;
+    return k < s.rot_dim ? to_f(x[k]) : 0.0f;
+}
+
 // Per row: rotates the heads' rotated query parts in place; a layer with keys of its own also norms the latent, rotates the shared
 // key part and puts both into the cache.
 template <typename T>
 __global__ void latent_prepare_kernel(T *__restrict__ proj, long long ld, const float2 *__restrict__ table, const float *__restrict__ norm_w, float eps,
-                                      const LatentShape s, int own_keys, const StepEntry *__restrict__ entries, const int *__restrict__ row_entry)
+                                      const LatentShape s, int own_keys, const StepEntry *__restrict__ entries, const int *__restrict__ row_entry, int row0)
 {
     __shared__ float red[32];
     grid_dependency_wait();
     grid_dependency_launch();
-    const int row = blockIdx.x;
+    const int row = row0 + blockIdx.x;
     const StepEntry e = entries[row_entry[row]];
     T *r = proj + row * ld;
     const float2 *cs = table + static_cast<long long>(row) * s.rot_half;
@@ -78,21 +87,12 @@ __global__ void latent_prepare_kernel(T *__restrict__ proj, long long ld, const 
     for (int i = threadIdx.x; i < s.rank_pitch; i += blockDim.x) dst[i] = from_f<T>(i < s.kv_rank ? to_f(d[i]) * inv * norm_w[i] : 0.0f);
     const T *kr = d + s.kv_rank;
     T *kd = dst + s.rank_pitch;
-    for (int k = threadIdx.x; k < s.row_pitch - s.rank_pitch; k += blockDim.x) {
-        float v = 0.0f;
-        if (k < s.rot_half)
-            v = to_f(kr[k]) * cs[k].x - to_f(kr[k + s.rot_half]) * cs[k].y;
-        else if (k < 2 * s.rot_half)
-            v = to_f(kr[k]) * cs[k - s.rot_half].x + to_f(kr[k - s.rot_half]) * cs[k - s.rot_half].y;
-        else if (k < s.rot_dim)
-            v = to_f(kr[k]);
-        kd[k] = from_f<T>(v);
-    }
+    for (int k = threadIdx.x; k < s.row_pitch - s.rank_pitch; k += blockDim.x) kd[k] = from_f<T>(rotated(kr, k, cs, s));
 }
 
 constexpr int kLatentWarps = 4;
 
-// Absorbed form, one block per (head, row): the query is mapped into the latent space, every warp goes through every fourth
+// Absorbed form for fp32 work, one block per (head, row): the query is mapped into the latent space, every warp goes through every fourth
 // visible position with a running maximum and sum, the warps' parts are merged, W_uv and the output gate are applied.
 // NR: cached row values per lane.  w_uk [heads * dim_pad][rank_pitch], w_uv [heads * v_pad][rank_pitch].
 template <typename T, int NR>

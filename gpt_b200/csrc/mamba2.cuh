@@ -22,11 +22,11 @@ template <typename T>
 __global__ void mamba_conv_kernel(T *__restrict__ xbc, int ld_xbc, float *__restrict__ dt, float *__restrict__ log_decay, const T *__restrict__ proj, long long ld_proj,
                                   const float *__restrict__ dt_raw, int ld_dt, const float *__restrict__ taps, const float *__restrict__ conv_b,
                                   const float *__restrict__ dt_bias, const float *__restrict__ a_log, const MambaShape s, const StepEntry *__restrict__ entries,
-                                  const int *__restrict__ row_entry, int conv_blocks)
+                                  const int *__restrict__ row_entry, int conv_blocks, int row0)
 {
     grid_dependency_wait();
     grid_dependency_launch();
-    const int row = blockIdx.y;
+    const int row = row0 + blockIdx.y;
     if (static_cast<int>(blockIdx.x) >= conv_blocks) {
         const int h = (blockIdx.x - conv_blocks) * blockDim.x + threadIdx.x;
         if (h < s.heads) {
@@ -106,6 +106,82 @@ __global__ void mamba_scan_kernel(float *__restrict__ y, const T *__restrict__ x
     }
     __syncthreads();
     for (int i = threadIdx.x; i < N * P; i += blockDim.x) state[i] = S[i];
+}
+
+constexpr int kStepCols = 32;   // value columns per block of the single-token kernel
+
+// One token: convolution, step size and recurrence in one launch.  One block per (head, 32 value columns, entry): a lane per column,
+// the eight warps share the state rows.  The convolution of B and C is computed by every block of the group; its inputs are
+// stored by the group's first.
+template <typename T>
+__global__ void __launch_bounds__(256)
+mamba_step_kernel(float *__restrict__ y, const T *__restrict__ proj, long long ld_proj, const float *__restrict__ dt_raw, int ld_dt, const float *__restrict__ taps,
+                  const float *__restrict__ conv_b, const float *__restrict__ dt_bias, const float *__restrict__ a_log, const float *__restrict__ d_skip, const MambaShape s,
+                  const StepEntry *__restrict__ entries)
+{
+    extern __shared__ float sm[];   // B [N] | C [N] | x [32] | partial sums [8][32]
+    const int P = s.vdim, N = s.state;
+    const int slices = (P + kStepCols - 1) / kStepCols;
+    const int h = blockIdx.x / slices, p0 = (blockIdx.x % slices) * kStepCols;
+    const int per_group = s.heads / s.groups, g = h / per_group;
+    float *x = sm + 2 * N, *part = x + kStepCols;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    grid_dependency_wait();
+    grid_dependency_launch();
+    const StepEntry e = entries[blockIdx.y];
+    const long long row = e.row0;
+    const int back = s.taps - 1;
+    T *conv = reinterpret_cast<T *>(e.slot + s.conv_state);
+    const T *old = conv + static_cast<long long>(e.parity) * back * s.channels;
+    T *next = conv + static_cast<long long>(e.parity ^ 1) * back * s.channels;
+    const bool owns_bc = p0 == 0 && h == g * per_group;
+    for (int i = threadIdx.x; i < 2 * N + kStepCols; i += blockDim.x) {
+        const bool is_x = i >= 2 * N;
+        if (is_x && p0 + i - 2 * N >= P) {
+            x[i - 2 * N] = 0.0f;
+            continue;
+        }
+        const int c = is_x ? h * P + p0 + i - 2 * N : i < N ? s.inner + g * N + i : s.inner + s.groups * N + g * N + i - N;
+        const T now = proj[row * ld_proj + s.inner + c];
+        float acc = conv_b[c];
+        for (int k = 0; k < back; ++k) {
+            const T v = old[static_cast<long long>(k) * s.channels + c];
+            acc = fmaf(taps[c * s.taps + k], to_f(v), acc);
+            if ((is_x || owns_bc) && k > 0) next[static_cast<long long>(k - 1) * s.channels + c] = v;
+        }
+        if ((is_x || owns_bc) && back > 0) next[static_cast<long long>(back - 1) * s.channels + c] = now;
+        acc = fmaf(taps[c * s.taps + back], to_f(now), acc);
+        sm[i] = to_f(from_f<T>(silu_f(acc)));   // rounded as the convolution of longer portions leaves it
+    }
+    const float step = softplus_f(dt_raw[row * ld_dt + h] + dt_bias[h]), keep = expf(-expf(a_log[h]) * step);
+    __syncthreads();
+    float *state = reinterpret_cast<float *>(e.slot + s.ssm_state) + static_cast<long long>(h) * N * P + p0 + lane;
+    float acc = 0.0f;
+    if (p0 + lane < P) {
+        const float xs = step * x[lane];
+        for (int n0 = warp; n0 < N; n0 += 64) {   // eight rows in flight
+            float v[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] = n0 + 8 * i < N ? state[static_cast<long long>(n0 + 8 * i) * P] : 0.0f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int n = n0 + 8 * i;
+                if (n < N) {
+                    v[i] = fmaf(keep, v[i], xs * sm[n]);
+                    state[static_cast<long long>(n) * P] = v[i];
+                    acc = fmaf(sm[N + n], v[i], acc);
+                }
+            }
+        }
+    }
+    part[warp * kStepCols + lane] = acc;
+    __syncthreads();
+    if (warp == 0 && p0 + lane < P) {
+        float v = d_skip[h] * x[lane];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v += part[i * kStepCols + lane];
+        y[row * s.inner + h * P + p0 + lane] = v;
+    }
 }
 
 // y * silu(z), then each of norm_groups parts divided by its own root mean square, times weight, as T [rows][ld_out].
