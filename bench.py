@@ -985,6 +985,182 @@ def run_attention(args):
     print(json.dumps(out), flush=True)
 
 
+# Decoder models whose layers have the proportions of real ones (random weights, three Mamba-2 layers to one of latent attention), and
+# the GPT-2 configuration of the same width, feed-forward width and number of layers.
+DECODER_SIZES = {
+    "w768": dict(width=768, ff=3072, heads=24, state=64, groups=1, att_heads=12, dim=64, rot_dim=32, vdim=64, kv_rank=256, side=64, layers=12, vocab=50304),
+    "w2048": dict(width=2048, ff=8192, heads=64, state=128, groups=8, att_heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, side=128, layers=8, vocab=50304),
+    "w4096": dict(width=4096, ff=14336, heads=128, state=128, groups=8, att_heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, side=256, layers=4, vocab=50304),
+}
+
+
+def decoder_folder(torch, dev, folder, z):
+    """Writes config.json and model.safetensors of a Budurax model of size z with random bf16 weights (generated on the GPU)."""
+    inner, bc = z["heads"] * 64, z["groups"] * z["state"]
+    W, layers = z["width"], []
+    shapes = [("embed", (z["vocab"], W)), ("side.embed", (z["vocab"], z["layers"] * z["side"]))]
+    for i in range(z["layers"]):
+        p = f"l{i}."
+        if i % 4 == 3:
+            rot = dict(base=500000.0, dims=z["rot_dim"], scaling=dict(factor=4.0, original=8192, fast=32.0, slow=1.0))
+            layers.append(dict(type="latent_attention", mlp=dict(kind="dense", ff=z["ff"]),
+                               mixer=dict(heads=z["att_heads"], dim=z["dim"], rot_dim=z["rot_dim"], vdim=z["vdim"], kv_rank=z["kv_rank"], scale=(z["dim"] + z["rot_dim"]) ** -0.5, rot=rot)))
+            H = z["att_heads"]
+            shapes += [(p + "mix.q", (H * (z["dim"] + z["rot_dim"]), W)), (p + "mix.dkv", (z["kv_rank"] + z["rot_dim"], W)), (p + "mix.dkv.norm", (z["kv_rank"],)),
+                       (p + "mix.uk", (H * z["dim"], z["kv_rank"])), (p + "mix.uv", (H * z["vdim"], z["kv_rank"])), (p + "mix.g", (H * z["vdim"], W)), (p + "mix.o", (W, H * z["vdim"]))]
+        else:
+            layers.append(dict(type="mamba2", mlp=dict(kind="dense", ff=z["ff"]),
+                               mixer=dict(heads=z["heads"], vdim=64, state=z["state"], groups=z["groups"], conv=4, norm_groups=z["groups"])))
+            shapes += [(p + "mix.in", (2 * inner + 2 * bc + z["heads"], W)), (p + "mix.conv", (inner + 2 * bc, 4)), (p + "mix.conv.b", (inner + 2 * bc,)), (p + "mix.dt_bias", (z["heads"],)),
+                       (p + "mix.A_log", (z["heads"],)), (p + "mix.D", (z["heads"],)), (p + "mix.norm", (inner,)), (p + "mix.o", (W, inner))]
+        shapes += [(p + "mlp.gate", (z["ff"], W)), (p + "mlp.up", (z["ff"], W)), (p + "mlp.down", (W, z["ff"])), (p + "shift", (W,)), (p + "dwa", (i + 2,)), (p + "side.gate", (z["side"], W)),
+                   (p + "side.proj", (W, z["side"])), (p + "side.norm", (W,))]
+        for n in ("norm1", "norm1b", "norm2", "norm2b"):
+            shapes += [(p + n, (W,)), (p + n + ".b", (W,))]
+    shapes += [("final.norm", (W,)), ("final.norm.b", (W,)), ("head", (z["vocab"], W))]
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(dict(architecture="Budurax", width=W, vocab=z["vocab"], norm=dict(eps=1e-5), token_side=dict(dim=z["side"]), layers=layers), f)
+    header, at = {}, 0
+    for name, shape in shapes:
+        n = 2
+        for d in shape:
+            n *= d
+        header[name] = dict(dtype="BF16", shape=list(shape), data_offsets=[at, at + n])
+        at += n
+    text = json.dumps(header).encode()
+    gen = torch.Generator(device=dev).manual_seed(1)
+    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
+        f.write(len(text).to_bytes(8, "little") + text)
+        for name, shape in shapes:
+            t = torch.randn(shape, device=dev, generator=gen) * (shape[1] ** -0.5 if len(shape) == 2 else 0.1)
+            if name.endswith("dwa"):
+                t[-1] += 1.0
+            if name.endswith("norm") or name[-6:-1] == ".norm" or name.endswith(("norm1b", "norm2b")):
+                t += 1.0
+            f.write(t.bfloat16().view(torch.int16).cpu().numpy().tobytes())
+    return at
+
+
+def decoder_record(torch, dev, sizes, prompts=(2048, 8192), context=1024, batches=(1, 8), steps=64, reps=3, gpt2=True):
+    """Prompt and decoding throughput of Budurax models (bf16) of real layer sizes through the public API (gpt_b200.serving.load_model:
+    step / generate, token ids from and to the host), and of GPT-2 (fp32, TF32 products) with the same width, feed-forward
+    width and number of layers: a forward pass over 8 x 1024 tokens, and its CUDA-graph-replayed decode step."""
+    import gpt_b200
+    from gpt_b200 import serving
+    out, launches = {}, 0
+    for name in sizes:
+        z = DECODER_SIZES[name]
+        rec = {"parameters_bytes": 0, "prompt": {}, "decode": {}}
+        with tempfile.TemporaryDirectory() as folder:
+            rec["parameters_bytes"] = decoder_folder(torch, dev, folder, z)
+            stream = torch.cuda.Stream()
+            model = serving.load_model(folder, "bfloat16", dev.index, stream.cuda_stream)
+        gen = torch.Generator().manual_seed(2)
+        l0 = model.launch_count()
+
+        def timed(fn):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            stream.synchronize()
+            e0.record(stream)
+            fn()
+            e1.record(stream)
+            e1.synchronize()
+            return e0.elapsed_time(e1)
+
+        for n in prompts:
+            tokens = torch.randint(0, z["vocab"], (n,), generator=gen).tolist()
+            times = []
+            for _ in range(reps + 1):
+                seq = model.open(n)
+                times.append(timed(lambda: model.step([(seq, tokens)], [n - 1])))
+                model.close(seq)
+            ms = statistics.median(times[1:])
+            rec["prompt"][str(n)] = dict(ms=ms, tokens_per_s=n / ms * 1e3)
+        for batch in batches:
+            seqs = [model.open(context + 4 * steps) for _ in range(batch)]
+            for s in seqs:
+                model.step([(s, torch.randint(0, z["vocab"], (context,), generator=gen).tolist())], [])
+            last = model.generate(seqs, [1] * batch, steps)[-1]          # eager step, capture, first replays
+            times = []
+            for _ in range(3):
+                e = timed(lambda: model.generate(seqs, [int(t) for t in last], steps))
+                times.append(e / steps)
+            ms = statistics.median(times)
+            rec["decode"][f"batch{batch}"] = dict(ms_per_step=ms, tokens_per_s=batch / ms * 1e3, context=context)
+            for s in seqs:
+                model.close(s)
+        launches += model.launch_count() - l0
+        model.close_model()
+        if gpt2:
+            rec["gpt2"] = decoder_gpt2(torch, dev, z, context, batches, steps, reps)
+        out[name] = rec
+    return dict(sizes=out, gpu_launches=int(launches))
+
+
+def decoder_gpt2(torch, dev, z, context, batches, steps, reps):
+    import gpt_b200
+    heads = z["width"] // 64
+    cfg = dict(max_seq_len=context + steps, vocab_size=z["vocab"], vocab_size_padded=z["vocab"], num_layers=z["layers"], num_heads=heads, d_model=z["width"], d_ffn=4 * z["width"])
+    stream = torch.cuda.Stream()
+    rec = {"d_ffn": cfg["d_ffn"]}
+    with torch.cuda.stream(stream):
+        m = gpt_b200.Model(cfg, dev.index, stream.cuda_stream, gpt_b200.MODE_TF32, use_grad=False)
+        m.init(0.0, 0.02)
+        m.set_option("decode_early_launch", 1)
+        tok = torch.randint(0, z["vocab"], (8, 1024), dtype=torch.int32, device=dev)
+        m.set_size(8, 1024)
+        ev = [torch.cuda.Event(enable_timing=True) for _ in range(2)]
+        times = []
+        for _ in range(reps + 1):
+            ev[0].record()
+            m.forward(tok)
+            ev[1].record()
+            stream.synchronize()
+            times.append(ev[0].elapsed_time(ev[1]))
+        ms = statistics.median(times[1:])
+        rec["prompt_8x1024"] = dict(ms=ms, tokens_per_s=8192 / ms * 1e3)
+        for batch in batches:
+            t1, logits = tok[:batch, 0].contiguous(), torch.empty(batch, z["vocab"], device=dev)
+            m.generate_begin(tok[:batch, :context].contiguous(), batch, context, context + steps)
+            m.generate_step(t1, logits)
+            stream.synchronize()
+            graph = torch.cuda.CUDAGraph()
+            m.generate_begin(tok[:batch, :context].contiguous(), batch, context, context + steps)
+            with torch.cuda.graph(graph, stream=stream):
+                m.generate_step(t1, logits)
+            graph.replay()
+            stream.synchronize()
+            ev[0].record()
+            for _ in range(steps - 2):
+                graph.replay()
+            ev[1].record()
+            stream.synchronize()
+            ms = ev[0].elapsed_time(ev[1]) / (steps - 2)
+            rec[f"decode_batch{batch}"] = dict(ms_per_step=ms, tokens_per_s=batch / ms * 1e3)
+            del graph
+        m.close()
+    return rec
+
+
+def run_decoder(args):
+    """--workload decoder: see decoder_record; the JSON `value` is the prompt throughput of the middle size at 8192 tokens."""
+    import torch
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    sampler = ClockSampler(0)
+    t_begin = time.time()
+    sizes = args.decoder_sizes.split(",")
+    rec = decoder_record(torch, dev, sizes, gpt2=not args.profile)
+    clocks = sampler.stop(t_begin, time.time())
+    main_rec = rec["sizes"]["w2048" if "w2048" in sizes else sizes[0]]["prompt"]["8192"]
+    out = dict(metric="decoder_prompt_tokens_per_s", value=main_rec["tokens_per_s"], unit="tokens/s", n_gpus=1, steps=3, warmup=1, ms_per_step=main_rec["ms"], higher_is_better=True,
+               scaling="weak", vs_baseline=None, dtype="bf16", data="synthetic", impl="ours",
+               config=dict(workload="Budurax decoder models with real layer sizes, random weights: prompts and CUDA-graph decoding through gpt_b200.serving; GPT-2 of equal width beside them",
+                           sizes={k: DECODER_SIZES[k] for k in sizes}, l2="weights and activations of a step (> 400 MB) exceed the 126 MB L2 at w2048 and w4096"),
+               sizes=rec["sizes"], gpu_launches=rec["gpu_launches"], clocks=clocks)
+    print(json.dumps(out), flush=True)
+
+
 def run_generate(args):
     """--workload generate: see generate_record; the JSON `value` is the batch-8 KV-cached figure."""
     import torch
@@ -1086,8 +1262,9 @@ def main():
     ap.add_argument("--cpu-rows", type=int, default=256, help="rows of the workload the cpu_baseline leg runs")
     ap.add_argument("--ref-rows", type=int, default=32, help="rows per step of the --impl reference arm")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--workload", choices=["ffn", "train", "decode", "generate", "attention"], default="ffn",
-                    help="ffn: BASELINE configs[1] (default); train: configs[3]; decode: configs[4] (linear layers of a decode step); generate: configs[4] end to end")
+    ap.add_argument("--workload", choices=["ffn", "train", "decode", "generate", "attention", "decoder"], default="ffn",
+                    help="ffn: BASELINE configs[1] (default); train: configs[3]; decode: configs[4] (linear layers of a decode step); generate: configs[4] end to end; decoder: Budurax models beside GPT-2 of equal width")
+    ap.add_argument("--decoder-sizes", default="w768,w2048,w4096", help="decoder workload: sizes to run")
     ap.add_argument("--global-batch", type=int, default=64, help="sequences per step over all GPUs (train workload); sequences of the attention workload")
     ap.add_argument("--m-per-gpu", type=int, default=M_PER_GPU, help="tokens per GPU (smaller for profiler captures)")
     ap.add_argument("--max-sms", type=int, default=0, help="SMs the GEMM kernels may occupy (0 = all; experiments)")
@@ -1114,6 +1291,8 @@ def main():
         run_attention(args)
     elif args.workload == "generate":
         run_generate(args)
+    elif args.workload == "decoder":
+        run_decoder(args)
     else:
         run_ours(args)
 

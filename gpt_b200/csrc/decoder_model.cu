@@ -695,12 +695,22 @@ private:
                 continue;
             }
             const int ld_xbc = pad_to(s.channels, 8), conv_blocks = (s.channels + 127) / 128, dt_blocks = (s.heads + 127) / 128;
-            RC_TRY(launch(mamba_conv_kernel<T>, dim3(conv_blocks + dt_blocks, run), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, proj_, ld, dt_raw, ld_dt, d.taps, d.conv_b, d.dt_bias, d.a_log, s,
-                          entries_, row_entry_, conv_blocks, row0));
+            if (s.channels % 8 == 0 && s.inner % 8 == 0 && s.taps >= 1 && s.taps <= 4) {
+                const auto conv8 = [&](auto kernel) {
+                    const int blocks = (s.channels / 8 + 127) / 128;
+                    return launch(kernel, dim3(blocks + 1, (run + kConvRows - 1) / kConvRows), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, proj_, ld, dt_raw, ld_dt, d.taps, d.conv_b, d.dt_bias,
+                                  d.a_log, s, entries_, row_entry_, blocks, row0, run);
+                };
+                RC_TRY(s.taps == 1 ? conv8(mamba_conv8_kernel<T, 1>) : s.taps == 2 ? conv8(mamba_conv8_kernel<T, 2>) : s.taps == 3 ? conv8(mamba_conv8_kernel<T, 3>)
+                                                                                                                                     : conv8(mamba_conv8_kernel<T, 4>));
+            } else {
+                RC_TRY(launch(mamba_conv_kernel<T>, dim3(conv_blocks + dt_blocks, run), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, proj_, ld, dt_raw, ld_dt, d.taps, d.conv_b, d.dt_bias, d.a_log, s,
+                              entries_, row_entry_, conv_blocks, row0));
+            }
             RC_TRY(k == 2 ? mamba_chunks(d, entry0, n, ld_xbc) : mamba_tokens(d, entry0, n, ld_xbc));
         }
         const int part = s.inner / s.norm_groups;
-        return launch(mamba_gated_norm_kernel<T>, dim3(rows, s.norm_groups), dim3(std::min(256, pad_to(part, 32))), size_t(part) * sizeof(float), act_, d.mix_out,
+        return launch(mamba_gated_norm_kernel<T>, dim3(rows, s.norm_groups), dim3(std::min(256, pad_to((part + 3) / 4, 32))), size_t(part) * sizeof(float), act_, d.mix_out,
                       static_cast<const float *>(ssm_y_), static_cast<const T *>(proj_), ld, static_cast<const float *>(d.mix_norm), s, static_cast<float>(c_.eps));
     }
 

@@ -108,6 +108,114 @@ __global__ void mamba_scan_kernel(float *__restrict__ y, const T *__restrict__ x
     for (int i = threadIdx.x; i < N * P; i += blockDim.x) state[i] = S[i];
 }
 
+__device__ __forceinline__ void load8(const __nv_bfloat16 *src, uint32_t (&w)[8])   // raw: 8 values in 4 words
+{
+    const uint4 v = *reinterpret_cast<const uint4 *>(src);
+    w[0] = v.x; w[1] = v.y; w[2] = v.z; w[3] = v.w;
+}
+__device__ __forceinline__ void load8(const float *src, uint32_t (&w)[8])
+{
+    const uint4 a = *reinterpret_cast<const uint4 *>(src), b = *reinterpret_cast<const uint4 *>(src + 4);
+    w[0] = a.x; w[1] = a.y; w[2] = a.z; w[3] = a.w; w[4] = b.x; w[5] = b.y; w[6] = b.z; w[7] = b.w;
+}
+template <typename T> __device__ __forceinline__ float raw8(const uint32_t (&w)[8], int i);
+template <> __device__ __forceinline__ float raw8<float>(const uint32_t (&w)[8], int i) { return __uint_as_float(w[i]); }
+template <> __device__ __forceinline__ float raw8<__nv_bfloat16>(const uint32_t (&w)[8], int i) { return i & 1 ? bf16_hi(w[i >> 1]) : bf16_lo(w[i >> 1]); }
+__device__ __forceinline__ void store8(__nv_bfloat16 *dst, const float (&v)[8])
+{
+    *reinterpret_cast<uint4 *>(dst) = make_uint4(ptx::pack_bf16x2(v[0], v[1]), ptx::pack_bf16x2(v[2], v[3]), ptx::pack_bf16x2(v[4], v[5]), ptx::pack_bf16x2(v[6], v[7]));
+}
+__device__ __forceinline__ void store8(float *dst, const float (&v)[8])
+{
+    store4(dst, make_float4(v[0], v[1], v[2], v[3]));
+    store4(dst + 4, make_float4(v[4], v[5], v[6], v[7]));
+}
+
+constexpr int kConvRows = 8;   // consecutive rows per thread
+
+// mamba_conv_kernel for channel counts and offsets that are multiples of 8: a thread slides over eight rows of eight channels with the
+// last inputs in registers.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+mamba_conv8_kernel(T *__restrict__ xbc, int ld_xbc, float *__restrict__ dt, float *__restrict__ log_decay, const T *__restrict__ proj, long long ld_proj, const float *__restrict__ dt_raw,
+                   int ld_dt, const float *__restrict__ taps, const float *__restrict__ conv_b, const float *__restrict__ dt_bias, const float *__restrict__ a_log, const MambaShape s,
+                   const StepEntry *__restrict__ entries, const int *__restrict__ row_entry, int conv_blocks, int row0, int rows)
+{
+    constexpr int BACK = TAPS - 1;
+    grid_dependency_wait();
+    grid_dependency_launch();
+    const int first = row0 + blockIdx.y * kConvRows, end = min(first + kConvRows, row0 + rows);
+    if (static_cast<int>(blockIdx.x) >= conv_blocks) {
+        for (int i = threadIdx.x; i < (end - first) * s.heads; i += blockDim.x) {
+            const long long row = first + i / s.heads;
+            const int h = i % s.heads;
+            const float step = softplus_f(dt_raw[row * ld_dt + h] + dt_bias[h]);
+            dt[row * s.heads + h] = step;
+            log_decay[row * s.heads + h] = -expf(a_log[h]) * step;
+        }
+        return;
+    }
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    if (c >= s.channels) return;
+    uint32_t in[kConvRows][8], window[BACK > 0 ? BACK : 1][8];   // window[k]: the input BACK - k steps back
+    const T *src = proj + s.inner + c;
+#pragma unroll
+    for (int i = 0; i < kConvRows; ++i)
+        if (first + i < end) load8(src + static_cast<long long>(first + i) * ld_proj, in[i]);
+    float w[8][TAPS], bias[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+        bias[j] = conv_b[c + j];
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) w[j][k] = taps[(c + j) * TAPS + k];
+    }
+    int entry = row_entry[first];
+    StepEntry e = entries[entry];
+    auto load_window = [&](int row) {   // the inputs before `row`
+        const T *old = reinterpret_cast<const T *>(e.slot + s.conv_state) + static_cast<long long>(e.parity) * BACK * s.channels + c;
+#pragma unroll
+        for (int k = 0; k < BACK; ++k) {
+            const int r = row - (BACK - k);
+            load8(r >= e.row0 ? src + static_cast<long long>(r) * ld_proj : old + static_cast<long long>(BACK + r - e.row0) * s.channels, window[k]);
+        }
+    };
+    load_window(first);
+#pragma unroll
+    for (int i = 0; i < kConvRows; ++i) {
+        const int row = first + i;
+        if (row >= end) break;
+        if (row == e.row0 + e.count) {
+            e = entries[++entry];
+            load_window(row);
+        }
+        float out[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            float acc = bias[j];
+#pragma unroll
+            for (int k = 0; k < BACK; ++k) acc = fmaf(w[j][k], raw8<T>(window[k], j), acc);
+            out[j] = silu_f(fmaf(w[j][BACK], raw8<T>(in[i], j), acc));
+        }
+        store8(xbc + static_cast<long long>(row) * ld_xbc + c, out);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+#pragma unroll
+            for (int k = 0; k + 1 < BACK; ++k) window[k][j] = window[k + 1][j];
+            if (BACK > 0) window[BACK > 0 ? BACK - 1 : 0][j] = in[i][j];
+        }
+        if (row == e.row0 + e.count - 1) {
+            T *next = reinterpret_cast<T *>(e.slot + s.conv_state) + static_cast<long long>(e.parity ^ 1) * BACK * s.channels + c;
+#pragma unroll
+            for (int k = 0; k < BACK; ++k) {
+                float v[8];
+#pragma unroll
+                for (int j = 0; j < 8; ++j) v[j] = raw8<T>(window[k], j);
+                store8(next + static_cast<long long>(k) * s.channels, v);
+            }
+        }
+    }
+}
+
 constexpr int kStepCols = 32;   // value columns per block of the single-token kernel
 
 // One token: convolution, step size and recurrence in one launch.  One block per (head, 32 value columns, entry): a lane per column,
@@ -196,6 +304,20 @@ __global__ void mamba_gated_norm_kernel(T *__restrict__ out, int ld_out, const f
     const long long row = blockIdx.x;
     const int part = s.inner / s.norm_groups, c0 = blockIdx.y * part;
     float ss = 0.0f;
+    if (part % 4 == 0) {   // y, z and the output are then aligned to four values
+        for (int i = 4 * threadIdx.x; i < part; i += 4 * blockDim.x) {
+            const float4 a = load4(y + row * s.inner + c0 + i), z = load4(proj + row * ld_proj + c0 + i);
+            const float4 v = make_float4(a.x * silu_f(z.x), a.y * silu_f(z.y), a.z * silu_f(z.z), a.w * silu_f(z.w));
+            store4(sm + i, v);
+            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+        const float inv = rsqrtf(block_sum(ss, red) / part + eps);
+        for (int i = 4 * threadIdx.x; i < part; i += 4 * blockDim.x) {
+            const float4 v = load4(sm + i), w = load4(weight + c0 + i);
+            store4(out + row * ld_out + c0 + i, make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w));
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < part; i += blockDim.x) {
         const float v = y[row * s.inner + c0 + i] * silu_f(to_f(proj[row * ld_proj + c0 + i]));
         sm[i] = v;
