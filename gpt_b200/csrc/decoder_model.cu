@@ -118,7 +118,7 @@ public:
                 d.mix_out = pad_to(s.inner, 8);
                 RC_TRY(matrix(file, &d.w_o, {{m + "o", W}}, s.inner, pitch_, d.mix_out));
                 s.conv_state = take(2 * size_t(s.taps - 1) * s.channels * sizeof(T));
-                s.ssm_state = take(size_t(a.heads) * a.state * a.vdim * sizeof(float));
+                s.ssm_state = take(2 * size_t(a.heads) * a.state * a.vdim * sizeof(float));
             } else {
                 const LatentConfig &a = l.latent;
                 LatentShape &s = d.latent;
@@ -246,6 +246,11 @@ public:
         if (!strcmp(key, "chunk_rows")) {   // Mamba-2: shortest portion that takes the chunked tensor-core form (0x7fffffff: none)
             if (value < 1) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "chunk_rows must be positive");
             chunk_rows_ = value;
+            return GPTB200_OK;
+        }
+        if (!strcmp(key, "segment_tokens")) {   // Mamba-2 prompts: tokens per segment (a multiple of 64)
+            if (value < kChunk || value % kChunk) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "segment_tokens must be a multiple of %d", kChunk);
+            segment_tokens_ = value;
             return GPTB200_OK;
         }
         if (!strcmp(key, "expand_rows")) {   // latent attention: shortest portion that takes the tensor-core form (0x7fffffff: none)
@@ -707,21 +712,37 @@ private:
                 RC_TRY(launch(mamba_conv_kernel<T>, dim3(conv_blocks + dt_blocks, run), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, proj_, ld, dt_raw, ld_dt, d.taps, d.conv_b, d.dt_bias, d.a_log, s,
                               entries_, row_entry_, conv_blocks, row0));
             }
-            RC_TRY(k == 2 ? mamba_chunks(d, entry0, n, ld_xbc) : mamba_tokens(d, entry0, n, ld_xbc));
+            RC_TRY(k == 2 ? mamba_chunks(d, parts, entry0, n, ld_xbc) : mamba_tokens(d, entry0, n, ld_xbc));
         }
         const int part = s.inner / s.norm_groups;
         return launch(mamba_gated_norm_kernel<T>, dim3(rows, s.norm_groups), dim3(std::min(256, pad_to((part + 3) / 4, 32))), size_t(part) * sizeof(float), act_, d.mix_out,
                       static_cast<const float *>(ssm_y_), static_cast<const T *>(proj_), ld, static_cast<const float *>(d.mix_norm), s, static_cast<float>(c_.eps));
     }
 
-    int mamba_chunks(const Layer &d, int entry0, int n, int ld_xbc)
+    int mamba_chunks(const Layer &d, const std::vector<Part> &parts, int entry0, int n, int ld_xbc)
     {
         if constexpr (kF32) {
             return mamba_tokens(d, entry0, n, ld_xbc);
         } else {
             const MambaShape &s = d.mamba;
-            return launch(mamba_chunk_kernel, dim3(s.heads * ((s.vdim + kChunkCols - 1) / kChunkCols), n), dim3(kChunkThreads), size_t(chunk_smem_bytes(s.state)), ssm_y_, xbc_, ld_xbc, dt_,
-                          decay_, d.d_skip, s, entries_ + entry0);
+            // segments that run side by side when a request alone would leave most of its time to one chunk after the other
+            int longest = 0;
+            for (int i = 0; i < n; ++i) longest = std::max(longest, parts[entry0 + i].count);
+            const int blocks = s.heads * ((s.vdim + kChunkCols - 1) / kChunkCols);
+            const int tokens = longest > segment_tokens_ + segment_tokens_ / 2 ? segment_tokens_ : pad_to(longest, kChunk);
+            const int segments = (longest + tokens - 1) / tokens;
+            const size_t smem = size_t(chunk_smem_bytes(s.state));
+            float *seg_state = nullptr, *seg_decay = nullptr;
+            if (segments > 1) {
+                const size_t pieces = size_t(n) * s.heads * segments;
+                RC_TRY(scratch(pieces * (size_t(s.state) * s.vdim + 1)));
+                seg_state = scratch_;
+                seg_decay = scratch_ + pieces * s.state * s.vdim;
+                RC_TRY(launch(mamba_chunk_kernel<true>, dim3(blocks, n, segments - 1), dim3(kChunkThreads), smem, ssm_y_, xbc_, ld_xbc, dt_, decay_, d.d_skip, s, entries_ + entry0, tokens,
+                              segments, seg_state, seg_decay));
+            }
+            return launch(mamba_chunk_kernel<false>, dim3(blocks, n, segments), dim3(kChunkThreads), smem, ssm_y_, xbc_, ld_xbc, dt_, decay_, d.d_skip, s, entries_ + entry0, tokens, segments,
+                          seg_state, seg_decay);
         }
     }
 
@@ -946,7 +967,7 @@ private:
     size_t fixed_state_ = 0, position_bytes_ = 0;
     std::vector<void *> weights_, work_;
     std::vector<Slot> slots_;
-    int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8;
+    int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8, segment_tokens_ = 512;
     T *expanded_ = nullptr;
     size_t expanded_count_ = 0;
     float *scratch_ = nullptr;

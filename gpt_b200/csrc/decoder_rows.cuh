@@ -44,6 +44,9 @@ __device__ __forceinline__ float4 load4(const __nv_bfloat16 *src)
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+// silu where its result is rounded to T: fast exponential and division (2 - 3 ulp of fp32) when that is bf16
+template <typename T> __device__ __forceinline__ float silu_t(float z) { return silu_f(z); }
+template <> __device__ __forceinline__ float silu_t<__nv_bfloat16>(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float gelu_f(float x) { return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x))); }
 

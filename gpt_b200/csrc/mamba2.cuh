@@ -1,8 +1,8 @@
 // Mamba-2 (state-space duality) layers: short causal convolution, step sizes and decays, the recurrence, the gated norm.
 //
 // A layer's projection row is [z: inner | x: inner | B: groups * state | C: groups * state] in T, its step sizes [heads] in fp32.  In a
-// sequence's slot: the convolution's last inputs [2][taps - 1][channels] in T (two copies, see StepEntry::parity) and
-// the state [heads][state][vdim] in fp32.  Steps, decays, exponentials, states and their sums are fp32.
+// sequence's slot: the convolution's last inputs [2][taps - 1][channels] in T and the state [2][heads][state][vdim] in fp32 (two copies
+// each, see StepEntry::parity).  Steps, decays, exponentials, states and their sums are fp32.
 #pragma once
 
 #include "decoder_rows.cuh"
@@ -50,7 +50,7 @@ __global__ void mamba_conv_kernel(T *__restrict__ xbc, int ld_xbc, float *__rest
     };
     float acc = conv_b[c];
     for (int k = s.taps - 1; k >= 0; --k) acc = fmaf(taps[c * s.taps + (back - k)], to_f(input(row, k)), acc);
-    xbc[static_cast<long long>(row) * ld_xbc + c] = from_f<T>(silu_f(acc));
+    xbc[static_cast<long long>(row) * ld_xbc + c] = from_f<T>(silu_t<T>(acc));
     if (row == e.row0 + e.count - 1) {
         T *next = state + static_cast<long long>(e.parity ^ 1) * back * s.channels;
         for (int k = 0; k < back; ++k) next[static_cast<long long>(back - 1 - k) * s.channels + c] = input(row, k);
@@ -72,7 +72,9 @@ __global__ void mamba_scan_kernel(float *__restrict__ y, const T *__restrict__ x
     grid_dependency_wait();
     grid_dependency_launch();
     float *state = reinterpret_cast<float *>(e.slot + s.ssm_state) + static_cast<long long>(h) * N * P;
-    for (int i = threadIdx.x; i < N * P; i += blockDim.x) S[i] = state[i];
+    const float *old_state = state + static_cast<long long>(e.parity) * s.heads * N * P;
+    state += static_cast<long long>(e.parity ^ 1) * s.heads * N * P;
+    for (int i = threadIdx.x; i < N * P; i += blockDim.x) S[i] = old_state[i];
     const int g = h / (s.heads / s.groups);
     const int p = threadIdx.x % P, q = threadIdx.x / P;
     const bool busy = q < lanes;
@@ -194,7 +196,7 @@ mamba_conv8_kernel(T *__restrict__ xbc, int ld_xbc, float *__restrict__ dt, floa
             float acc = bias[j];
 #pragma unroll
             for (int k = 0; k < BACK; ++k) acc = fmaf(w[j][k], raw8<T>(window[k], j), acc);
-            out[j] = silu_f(fmaf(w[j][BACK], raw8<T>(in[i], j), acc));
+            out[j] = silu_t<T>(fmaf(w[j][BACK], raw8<T>(in[i], j), acc));
         }
         store8(xbc + static_cast<long long>(row) * ld_xbc + c, out);
 #pragma unroll
@@ -259,18 +261,20 @@ mamba_step_kernel(float *__restrict__ y, const T *__restrict__ proj, long long l
         }
         if ((is_x || owns_bc) && back > 0) next[static_cast<long long>(back - 1) * s.channels + c] = now;
         acc = fmaf(taps[c * s.taps + back], to_f(now), acc);
-        sm[i] = to_f(from_f<T>(silu_f(acc)));   // rounded as the convolution of longer portions leaves it
+        sm[i] = to_f(from_f<T>(silu_t<T>(acc)));   // rounded as the convolution of longer portions leaves it
     }
     const float step = softplus_f(dt_raw[row * ld_dt + h] + dt_bias[h]), keep = expf(-expf(a_log[h]) * step);
     __syncthreads();
     float *state = reinterpret_cast<float *>(e.slot + s.ssm_state) + static_cast<long long>(h) * N * P + p0 + lane;
+    const float *old_state = state + static_cast<long long>(e.parity) * s.heads * N * P;
+    state += static_cast<long long>(e.parity ^ 1) * s.heads * N * P;
     float acc = 0.0f;
     if (p0 + lane < P) {
         const float xs = step * x[lane];
         for (int n0 = warp; n0 < N; n0 += 64) {   // eight rows in flight
             float v[8];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) v[i] = n0 + 8 * i < N ? state[static_cast<long long>(n0 + 8 * i) * P] : 0.0f;
+            for (int i = 0; i < 8; ++i) v[i] = n0 + 8 * i < N ? old_state[static_cast<long long>(n0 + 8 * i) * P] : 0.0f;
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 const int n = n0 + 8 * i;
@@ -307,7 +311,7 @@ __global__ void mamba_gated_norm_kernel(T *__restrict__ out, int ld_out, const f
     if (part % 4 == 0) {   // y, z and the output are then aligned to four values
         for (int i = 4 * threadIdx.x; i < part; i += 4 * blockDim.x) {
             const float4 a = load4(y + row * s.inner + c0 + i), z = load4(proj + row * ld_proj + c0 + i);
-            const float4 v = make_float4(a.x * silu_f(z.x), a.y * silu_f(z.y), a.z * silu_f(z.z), a.w * silu_f(z.w));
+            const float4 v = make_float4(a.x * silu_t<T>(z.x), a.y * silu_t<T>(z.y), a.z * silu_t<T>(z.z), a.w * silu_t<T>(z.w));
             store4(sm + i, v);
             ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
         }
@@ -319,7 +323,7 @@ __global__ void mamba_gated_norm_kernel(T *__restrict__ out, int ld_out, const f
         return;
     }
     for (int i = threadIdx.x; i < part; i += blockDim.x) {
-        const float v = y[row * s.inner + c0 + i] * silu_f(to_f(proj[row * ld_proj + c0 + i]));
+        const float v = y[row * s.inner + c0 + i] * silu_t<T>(to_f(proj[row * ld_proj + c0 + i]));
         sm[i] = v;
         ss = fmaf(v, v, ss);
     }
