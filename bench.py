@@ -1092,9 +1092,66 @@ def decoder_record(torch, dev, sizes, prompts=(2048, 8192), context=1024, batche
         launches += model.launch_count() - l0
         model.close_model()
         if gpt2:
+            rec["linear"] = decoder_linears(torch, dev, z)
             rec["gpt2"] = decoder_gpt2(torch, dev, z, context, batches, steps, reps)
         out[name] = rec
     return dict(sizes=out, gpu_launches=int(launches))
+
+
+def decoder_linears(torch, dev, z, rows=(1, 8, 4096), steps=10):
+    """The four large products of a layer pair (in_proj / o of Mamba-2, gated up, down) through gptb200_linear_bf16: GB/s of weight stream for
+    few rows (CUDA-graph replay over weight sets larger than L2, as decode_record does for GPT-2), TFLOP/s for prompts."""
+    import ctypes
+    import gpt_b200
+    from gpt_b200 import decoder
+    lib = decoder.load_library()
+    stream = torch.cuda.Stream()
+    be = gpt_b200.Backend(dev.index, stream.cuda_stream)
+    be.set_option("decode_early_launch", 1)
+    inner = z["heads"] * 64
+    n_in = 2 * inner + 2 * z["groups"] * z["state"] + z["heads"]
+    shapes = [("in", (n_in + 31) // 32 * 32, z["width"], 1), ("o", z["width"], inner, 0), ("glu", 2 * z["ff"], z["width"], 2), ("down", z["width"], z["ff"], 0)]
+    per_set = sum(2 * n * k for _, n, k, _ in shapes)
+    sets = max(2, -(-400_000_000 // per_set))
+    out = {}
+    with torch.cuda.stream(stream):
+        w = [{name: torch.empty(n, k, device=dev, dtype=torch.bfloat16).normal_(0, k ** -0.5) for name, n, k, _ in shapes} for _ in range(sets)]
+        for m in rows:
+            x = torch.randn(m, max(z["width"], inner, z["ff"]), device=dev).bfloat16()
+            y = torch.empty(m, max(n_in + 32, 2 * z["ff"]), device=dev)
+
+            def call(s, name, n, k, kind):
+                rc = lib.gptb200_linear_bf16(be.handle, kind, ctypes.c_void_p(y.data_ptr()), n // 2 if kind == 2 else n, ctypes.c_void_p(x.data_ptr()), k,
+                                             ctypes.c_void_p(w[s][name].data_ptr()), m, n, k, None, 1 << 30, 0, None, None, 0)
+                assert rc == 0
+
+            def run(only=None):
+                for s in range(sets):
+                    for name, n, k, kind in shapes:
+                        if only in (None, name):
+                            call(s, name, n, k, kind)
+            rec = {}
+            for only in ([None] if m <= 8 else []) + [n for n, *_ in shapes]:
+                run(only)
+                stream.synchronize()
+                graph = torch.cuda.CUDAGraph()
+                with torch.cuda.graph(graph, stream=stream):
+                    run(only)
+                graph.replay()
+                stream.synchronize()
+                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                e0.record()
+                for _ in range(steps):
+                    graph.replay()
+                e1.record()
+                stream.synchronize()
+                us = e0.elapsed_time(e1) * 1e3 / steps / sets
+                todo = [(n, k) for name, n, k, _ in shapes if only in (None, name)]
+                rec[only or "all"] = dict(us=us, gbs=sum(2 * n * k for n, k in todo) / us * 1e-3) if m <= 8 else dict(us=us, tflops=sum(2.0 * m * n * k for n, k in todo) / us * 1e-6)
+                del graph
+            out[f"rows{m}"] = rec
+    be.close()
+    return out
 
 
 def decoder_gpt2(torch, dev, z, context, batches, steps, reps):

@@ -110,6 +110,7 @@ public:
                 const int rows = a.inner() + s.channels;
                 RC_TRY(matrix(file, &d.w_in, {{m + "in", rows + a.heads}}, W, d.proj_n, pitch_, [&](int r) { return r < rows ? r : d.proj_cols + r - rows; }));
                 RC_TRY(vector(file, &d.taps, m + "conv", s.channels * s.taps, 0, {s.channels, s.taps}));
+                RC_TRY(transposed(file, &d.taps_t, m + "conv", s.channels, s.taps));
                 RC_TRY(vector(file, &d.conv_b, m + "conv.b", s.channels));
                 RC_TRY(vector(file, &d.dt_bias, m + "dt_bias", a.heads));
                 RC_TRY(vector(file, &d.a_log, m + "A_log", a.heads));
@@ -394,7 +395,7 @@ private:
         T *w_in = nullptr, *w_o = nullptr;
         int proj_n = 0, proj_cols = 0, mix_out = 0;
         MambaShape mamba{};
-        float *taps = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *a_log = nullptr, *d_skip = nullptr, *mix_norm = nullptr;
+        float *taps = nullptr, *taps_t = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *a_log = nullptr, *d_skip = nullptr, *mix_norm = nullptr;
         LatentShape latent{};
         T *w_uk = nullptr, *w_uv = nullptr;
         bool own_keys = false;
@@ -479,6 +480,14 @@ private:
         const TensorView &t = tensor(f, name, shape.empty() ? std::vector<long long>{n} : shape);
         std::vector<float> host(std::max(n, padded), 0.0f);
         for (int i = 0; i < n; ++i) host[i] = element(t, i);
+        return to_device(out, host);
+    }
+    int transposed(const SafeTensors &f, float **out, const std::string &name, int rows, int cols)
+    {
+        const TensorView &t = tensor(f, name, {rows, cols});
+        std::vector<float> host(size_t(rows) * cols);
+        for (int i = 0; i < rows; ++i)
+            for (int j = 0; j < cols; ++j) host[size_t(j) * rows + i] = element(t, 1LL * i * cols + j);
         return to_device(out, host);
     }
     int norm(const SafeTensors &f, Norm *out, const std::string &name)
@@ -640,7 +649,8 @@ private:
         }
     }
 
-    int row_threads() const { return std::min(256, std::max(32, pad_to(pitch_ / 4, 32))); }
+    // threads per row of the stream: with few rows a row is spread wider
+    int row_threads(int rows) const { return std::min(rows <= 2 * ctx_->num_sms ? 1024 : 256, std::max(32, pad_to(pitch_ / 4, 32))); }
 
     int layer_begin(int rows, int layer, const T *h, const int *row_list)
     {
@@ -668,7 +678,7 @@ private:
         b.h = const_cast<T *>(h);
         b.entries = entries_; b.row_entry = row_entry_; b.row_list = row_list;
         b.tile = rows <= 512 || !b.shift ? 1 : rows <= 2048 ? 4 : 8;
-        return launch(layer_begin_kernel<T>, dim3((rows + b.tile - 1) / b.tile), dim3(row_threads()), 2 * size_t(pitch_) * sizeof(float), b);
+        return launch(layer_begin_kernel<T>, dim3((rows + b.tile - 1) / b.tile), dim3(row_threads(rows)), 2 * size_t(pitch_) * sizeof(float), b);
     }
 
     int mamba(const Layer &d, const std::vector<Part> &parts, int rows)
@@ -703,7 +713,7 @@ private:
             if (s.channels % 8 == 0 && s.inner % 8 == 0 && s.taps >= 1 && s.taps <= 4) {
                 const auto conv8 = [&](auto kernel) {
                     const int blocks = (s.channels / 8 + 127) / 128;
-                    return launch(kernel, dim3(blocks + 1, (run + kConvRows - 1) / kConvRows), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, proj_, ld, dt_raw, ld_dt, d.taps, d.conv_b, d.dt_bias,
+                    return launch(kernel, dim3(blocks + 1, (run + kConvRows - 1) / kConvRows), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, proj_, ld, dt_raw, ld_dt, d.taps_t, d.conv_b, d.dt_bias,
                                   d.a_log, s, entries_, row_entry_, blocks, row0, run);
                 };
                 RC_TRY(s.taps == 1 ? conv8(mamba_conv8_kernel<T, 1>) : s.taps == 2 ? conv8(mamba_conv8_kernel<T, 2>) : s.taps == 3 ? conv8(mamba_conv8_kernel<T, 3>)
@@ -912,7 +922,7 @@ private:
     int kernels(const std::vector<Part> &parts, int rows, int n_want)
     {
         const float eps = static_cast<float>(c_.eps);
-        RC_TRY(launch(embed_rows_kernel<T>, dim3(rows), dim3(row_threads()), 0, states_, static_cast<const T *>(embed_), static_cast<const int *>(tokens_), pitch_));
+        RC_TRY(launch(embed_rows_kernel<T>, dim3(rows), dim3(row_threads(rows)), 0, states_, static_cast<const T *>(embed_), static_cast<const int *>(tokens_), pitch_));
         for (const Rotary &r : rotaries_)
             RC_TRY(launch(rotary_table_kernel, dim3((rows * (r.config.dims / 2) + 127) / 128), dim3(128), 0, table_ + r.table, static_cast<const double *>(r.freq), r.config.dims / 2, r.gain,
                           entries_, row_entry_, rows));
@@ -923,7 +933,7 @@ private:
             RC_TRY(c_.layers[i].kind == MixerKind::Mamba2 ? mamba(d, parts, rows) : latent(d, parts, rows));
             RC_TRY(linear_f32(y_, act_, d.w_o, rows, pitch_, d.mix_out));
             const size_t smem = size_t(pitch_) * sizeof(float);
-            RC_TRY(launch(sublayer_end_kernel<T>, dim3(rows), dim3(row_threads()), smem, x, static_cast<const float *>(y_), static_cast<const float *>(d.norm1b.w),
+            RC_TRY(launch(sublayer_end_kernel<T>, dim3(rows), dim3(row_threads(rows)), smem, x, static_cast<const float *>(y_), static_cast<const float *>(d.norm1b.w),
                           static_cast<const float *>(d.norm1b.b), static_cast<const float *>(d.norm2.w), static_cast<const float *>(d.norm2.b), h_, c_.width, pitch_, eps));
             if (d.ff) {
                 if constexpr (kF32) {
@@ -935,7 +945,7 @@ private:
                     RC_TRY(run_linear_bf16(ctx_, c));
                 }
                 RC_TRY(linear_f32(y_, act_, d.w_down, rows, pitch_, d.ff));
-                RC_TRY(launch(sublayer_end_kernel<T>, dim3(rows), dim3(row_threads()), smem, x, static_cast<const float *>(y_), static_cast<const float *>(d.norm2b.w),
+                RC_TRY(launch(sublayer_end_kernel<T>, dim3(rows), dim3(row_threads(rows)), smem, x, static_cast<const float *>(y_), static_cast<const float *>(d.norm2b.w),
                               static_cast<const float *>(d.norm2b.b), static_cast<const float *>(nullptr), static_cast<const float *>(nullptr), h_, c_.width, pitch_, eps));
             }
             if (d.side_gate) {

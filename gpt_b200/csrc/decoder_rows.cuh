@@ -59,8 +59,9 @@ __device__ __forceinline__ float block_sum(float v, float *red)
     __syncthreads();   // the previous use of `red` is over
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
     __syncthreads();
-    float s = 0.0f;
-    for (int i = 0; i < warps; ++i) s += red[i];
+    float s = (threadIdx.x & 31) < warps ? red[threadIdx.x & 31] : 0.0f;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
     return s;
 }
 

@@ -1,9 +1,10 @@
 // Products of up to eight rows with a bf16 weight matrix stored [n][k]: out[m][n] = x[m][k] . w[n][k], fp32 accumulation, with the
-// outputs of the bf16 tensor-core form (OutKind).  The weights are streamed once: a warp takes two weight rows at a time, 512
-// contiguous bytes of each per step, the activations come from shared memory.
+// outputs of the bf16 tensor-core form (OutKind).  The weights are streamed once and the activations come from shared memory.
+// One row: a warp takes two weight rows at a time, 512 contiguous bytes of each per step, fp32 FMAs.  Two to eight rows:
+// gemv_bf16_mma_kernel.
 //
-// The kernel may be launched with programmatic stream serialization: it requests its first weights while its predecessor on
-// the stream still runs and touches activations and outputs only after griddepcontrol.wait (weights are never written
+// The kernels may be launched with programmatic stream serialization: they request their first weights while their predecessor on
+// the stream still runs and touch activations and outputs only after griddepcontrol.wait (weights are never written
 // by a kernel of a step).
 #pragma once
 
@@ -80,11 +81,10 @@ __device__ __forceinline__ void gemv_pair(int i, int out_kind, int &ra, int &rb)
     }
 }
 
-template <int MR>
-__global__ void __launch_bounds__(kGemvThreads)
+static __global__ void __launch_bounds__(kGemvThreads)
 gemv_bf16_kernel(const GemvParams p)
 {
-    extern __shared__ uint4 gemv_x[];   // [MR][K / 8]
+    extern __shared__ uint4 gemv_x[];   // [K / 8]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int chunks = p.K >> 3;
     const int pairs = p.out_kind == OUT_GLU ? p.N / 2 : (p.N + 1) / 2;
@@ -107,27 +107,19 @@ gemv_bf16_kernel(const GemvParams p)
     if (pair < pairs) fetch(pair, 0);
     grid_dependency_wait();
     grid_dependency_launch();
-    for (int i = threadIdx.x; i < MR * chunks; i += kGemvThreads) {
-        const int m = i / chunks, c = i % chunks;
-        gemv_x[i] = m < p.M ? *(reinterpret_cast<const uint4 *>(p.x + m * p.ldx) + c) : make_uint4(0u, 0u, 0u, 0u);
-    }
+    for (int i = threadIdx.x; i < chunks; i += kGemvThreads) gemv_x[i] = *(reinterpret_cast<const uint4 *>(p.x) + i);
     __syncthreads();
     for (; pair < pairs; pair += stride) {
-        float sa[MR], sb[MR];
-#pragma unroll
-        for (int m = 0; m < MR; ++m) sa[m] = sb[m] = 0.0f;
+        float sa = 0.0f, sb = 0.0f;
         for (int c0 = 0; c0 < chunks; c0 += 32 * kGemvUnroll) {
             if (c0 > 0) fetch(pair, c0);
 #pragma unroll
             for (int u = 0; u < kGemvUnroll; ++u) {
                 const int c = c0 + u * 32 + lane;
                 if (c < chunks) {
-#pragma unroll
-                    for (int m = 0; m < MR; ++m) {
-                        const uint4 xv = gemv_x[m * chunks + c];
-                        sa[m] = dot8(wa[u], xv, sa[m]);
-                        sb[m] = dot8(wb[u], xv, sb[m]);
-                    }
+                    const uint4 xv = gemv_x[c];
+                    sa = dot8(wa[u], xv, sa);
+                    sb = dot8(wb[u], xv, sb);
                 }
             }
         }
@@ -136,20 +128,106 @@ gemv_bf16_kernel(const GemvParams p)
         int ra, rb;
         gemv_pair(done, p.out_kind, ra, rb);
 #pragma unroll
-        for (int m = 0; m < MR; ++m) {
+        for (int o = 16; o > 0; o >>= 1) {
+            sa += __shfl_xor_sync(0xffffffffu, sa, o);
+            sb += __shfl_xor_sync(0xffffffffu, sb, o);
+        }
+        if (lane == 0) {
+            gemv_emit(p, 0, ra, sa, sb);
+            if (p.out_kind != OUT_GLU && rb < p.N) gemv_emit(p, 0, rb, sb, 0.0f);
+        }
+    }
+}
+
+// Two to eight rows: the same stream of weights as the A operand of m16n8k16 products (16 weight rows, up to eight rows of x).  A
+// block takes TILES x 16 weight rows (OUT_GLU: 16 gate rows and their 16 up rows) and its eight warps share k.  The order of k inside a block
+// of 32 is permuted alike on both sides so that a lane loads 16 contiguous bytes of a row: piece c of a block (8 values) feeds
+// two products, values 0-3 the first and 4-7 the second.
+constexpr int kGemvMmaUnroll = 4;   // blocks of 32 k in flight per warp
+
+__device__ __forceinline__ void gemv_mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1)
+{
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+__host__ __device__ inline int gemv_mma_pitch(int k) { return (k + 31) / 32 * 64 + ((k + 31) / 32 % 2 == 0 ? 64 : 0); }   // bytes, an odd multiple of 64
+
+template <int TILES>
+__global__ void __launch_bounds__(kGemvThreads)
+gemv_bf16_mma_kernel(const GemvParams p)
+{
+    extern __shared__ __align__(16) uint8_t gemv_sm[];   // x [M][pitch], then sums [8 warps][TILES * 16][8]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int g = lane >> 2, c = lane & 3;
+    const int pitch = gemv_mma_pitch(p.K);
+    float *sums = reinterpret_cast<float *>(gemv_sm + p.M * pitch);
+    // weight rows of the block's tiles
+    int row[TILES];
 #pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                sa[m] += __shfl_xor_sync(0xffffffffu, sa[m], o);
-                sb[m] += __shfl_xor_sync(0xffffffffu, sb[m], o);
+    for (int t = 0; t < TILES; ++t)
+        row[t] = p.out_kind == OUT_GLU ? (blockIdx.x >> 1) * 64 + (blockIdx.x & 1) * 16 + t * 32 : (blockIdx.x * TILES + t) * 16;
+    const int blocks = (p.K + 31) / 32, per_warp = (blocks + 7) / 8;
+    const int first = warp * per_warp, end = min(blocks, first + per_warp);
+    uint4 wv[kGemvMmaUnroll][TILES][2];
+    auto fetch = [&](int blk) {
+#pragma unroll
+        for (int u = 0; u < kGemvMmaUnroll; ++u) {
+            const int k = (blk + u) * 32 + c * 8;
+#pragma unroll
+            for (int t = 0; t < TILES; ++t)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const int r = row[t] + g + 8 * half;
+                    wv[u][t][half] = blk + u < end && k < p.K && r < p.N ? __ldg(reinterpret_cast<const uint4 *>(p.w + static_cast<long long>(r) * p.K + k)) : make_uint4(0u, 0u, 0u, 0u);
+                }
+        }
+    };
+    fetch(first);
+    grid_dependency_wait();
+    grid_dependency_launch();
+    const int pieces = pitch / 16;
+    for (int i = threadIdx.x; i < p.M * pieces; i += kGemvThreads) {
+        const int m = i / pieces, q = i % pieces;
+        *reinterpret_cast<uint4 *>(gemv_sm + m * pitch + q * 16) = q * 8 < p.K ? *reinterpret_cast<const uint4 *>(p.x + m * p.ldx + q * 8) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    __syncthreads();
+    float acc[TILES][4] = {};
+    const bool live = g < p.M;   // this lane's row of x
+    const uint8_t *xs = gemv_sm + (live ? g : 0) * pitch + c * 16;
+    for (int blk = first; blk < end; blk += kGemvMmaUnroll) {
+        if (blk > first) fetch(blk);
+#pragma unroll
+        for (int u = 0; u < kGemvMmaUnroll; ++u) {
+            if (blk + u >= end) continue;
+            uint4 x = *reinterpret_cast<const uint4 *>(xs + (blk + u) * 64);
+            if (!live) x = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+            for (int t = 0; t < TILES; ++t) {
+                const uint4 a = wv[u][t][0], b = wv[u][t][1];
+                gemv_mma_bf16(acc[t], a.x, b.x, a.y, b.y, x.x, x.y);
+                gemv_mma_bf16(acc[t], a.z, b.z, a.w, b.w, x.z, x.w);
             }
         }
+    }
 #pragma unroll
-        for (int m = 0; m < MR; ++m) {
-            if (m < p.M && lane == m) {
-                gemv_emit(p, m, ra, sa[m], sb[m]);
-                if (p.out_kind != OUT_GLU && rb < p.N) gemv_emit(p, m, rb, sb[m], 0.0f);
-            }
+    for (int t = 0; t < TILES; ++t)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) sums[(warp * TILES * 16 + t * 16 + g + (i >> 1) * 8) * 8 + 2 * c + (i & 1)] = acc[t][i];
+    __syncthreads();
+    const int outputs = p.out_kind == OUT_GLU ? 128 : TILES * 128;
+    for (int i = threadIdx.x; i < outputs; i += kGemvThreads) {
+        const int r = i >> 3, m = i & 7;
+        if (m >= p.M) continue;
+        float v = 0.0f, up = 0.0f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) {
+            v += sums[(w * TILES * 16 + r) * 8 + m];
+            if (TILES == 2 && p.out_kind == OUT_GLU) up += sums[(w * TILES * 16 + 16 + r) * 8 + m];
         }
+        const int n = p.out_kind == OUT_GLU ? row[0] + r : blockIdx.x * TILES * 16 + r;
+        if (n < p.N) gemv_emit(p, m, n, v, up);
     }
 }
 

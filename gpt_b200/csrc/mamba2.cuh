@@ -136,11 +136,11 @@ __device__ __forceinline__ void store8(float *dst, const float (&v)[8])
 constexpr int kConvRows = 8;   // consecutive rows per thread
 
 // mamba_conv_kernel for channel counts and offsets that are multiples of 8: a thread slides over eight rows of eight channels with the
-// last inputs in registers.
+// last inputs in registers.  taps_t [taps][channels].
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 4)
 mamba_conv8_kernel(T *__restrict__ xbc, int ld_xbc, float *__restrict__ dt, float *__restrict__ log_decay, const T *__restrict__ proj, long long ld_proj, const float *__restrict__ dt_raw,
-                   int ld_dt, const float *__restrict__ taps, const float *__restrict__ conv_b, const float *__restrict__ dt_bias, const float *__restrict__ a_log, const MambaShape s,
+                   int ld_dt, const float *__restrict__ taps_t, const float *__restrict__ conv_b, const float *__restrict__ dt_bias, const float *__restrict__ a_log, const MambaShape s,
                    const StepEntry *__restrict__ entries, const int *__restrict__ row_entry, int conv_blocks, int row0, int rows)
 {
     constexpr int BACK = TAPS - 1;
@@ -164,13 +164,14 @@ mamba_conv8_kernel(T *__restrict__ xbc, int ld_xbc, float *__restrict__ dt, floa
 #pragma unroll
     for (int i = 0; i < kConvRows; ++i)
         if (first + i < end) load8(src + static_cast<long long>(first + i) * ld_proj, in[i]);
-    float w[8][TAPS], bias[8];
+    float w[TAPS][8], bias[8];
+    auto vec8 = [&](const float *from, float (&to)[8]) {
+        const float4 a = __ldg(reinterpret_cast<const float4 *>(from)), b = __ldg(reinterpret_cast<const float4 *>(from + 4));
+        to[0] = a.x; to[1] = a.y; to[2] = a.z; to[3] = a.w; to[4] = b.x; to[5] = b.y; to[6] = b.z; to[7] = b.w;
+    };
+    vec8(conv_b + c, bias);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-        bias[j] = conv_b[c + j];
-#pragma unroll
-        for (int k = 0; k < TAPS; ++k) w[j][k] = taps[(c + j) * TAPS + k];
-    }
+    for (int k = 0; k < TAPS; ++k) vec8(taps_t + static_cast<long long>(k) * s.channels + c, w[k]);
     int entry = row_entry[first];
     StepEntry e = entries[entry];
     auto load_window = [&](int row) {   // the inputs before `row`
@@ -195,8 +196,8 @@ mamba_conv8_kernel(T *__restrict__ xbc, int ld_xbc, float *__restrict__ dt, floa
         for (int j = 0; j < 8; ++j) {
             float acc = bias[j];
 #pragma unroll
-            for (int k = 0; k < BACK; ++k) acc = fmaf(w[j][k], raw8<T>(window[k], j), acc);
-            out[j] = silu_t<T>(fmaf(w[j][BACK], raw8<T>(in[i], j), acc));
+            for (int k = 0; k < BACK; ++k) acc = fmaf(w[k][j], raw8<T>(window[k], j), acc);
+            out[j] = silu_t<T>(fmaf(w[BACK][j], raw8<T>(in[i], j), acc));
         }
         store8(xbc + static_cast<long long>(row) * ld_xbc + c, out);
 #pragma unroll
