@@ -1098,7 +1098,7 @@ def decoder_record(torch, dev, sizes, prompts=(2048, 8192), context=1024, batche
     return dict(sizes=out, gpu_launches=int(launches))
 
 
-def decoder_linears(torch, dev, z, rows=(1, 8, 4096), steps=10):
+def decoder_linears(torch, dev, z, rows=(1, 8, 8192), steps=10):
     """The four large products of a layer pair (in_proj / o of Mamba-2, gated up, down) through gptb200_linear_bf16: GB/s of weight stream for
     few rows (CUDA-graph replay over weight sets larger than L2, as decode_record does for GPT-2), TFLOP/s for prompts."""
     import ctypes

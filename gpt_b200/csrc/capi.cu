@@ -736,7 +736,7 @@ int run_linear_bf16_impl(gptb200_ctx *ctx, const Bf16Linear &c)
     if (c.K <= 0 || c.K % 8 || c.lda % 8 || !aligned16(c.a) || !aligned16(c.w) || !aligned16(c.out) || (c.out_kind == OUT_GLU && c.N % 64) ||
         (c.out_kind == OUT_BF16 && c.tail_col % 32 && c.tail_col < c.N) || (c.out_kind == OUT_GELU_MUL && (c.N % 8 || c.factor_pitch % 8 || !aligned16(c.factor))))
         return fail(ctx, GPTB200_ERR_INVALID_ARG, "bf16 product: sizes or alignment (M=%d N=%d K=%d lda=%lld kind=%d)", c.M, c.N, c.K, c.lda, c.out_kind);
-    if (c.M <= ctx->gemv_rows && size_t(c.M) * gemv_mma_pitch(c.K) + 8 * 32 * 8 * 4 <= 200 * 1024) {
+    if (c.M <= ctx->gemv_rows && (c.M > 1 || size_t(c.K) * 2 <= 200 * 1024)) {
         GemvParams g{c.M, c.N, c.K, static_cast<const uint16_t *>(c.a), c.lda, static_cast<const uint16_t *>(c.w), c.out_kind, c.out, c.ldo, c.tail, c.tail_col, c.tail_pitch,
                      static_cast<const uint16_t *>(c.factor), c.factor_rows, c.factor_pitch};
         if (c.M == 1) {
@@ -744,9 +744,8 @@ int run_linear_bf16_impl(gptb200_ctx *ctx, const Bf16Linear &c)
             return launch_gemv(ctx, gemv_bf16_kernel, g, std::max(1, std::min((pairs + per_cta - 1) / per_cta, ctx->num_sms * 4)), size_t(c.K) * 2);
         }
         const int tiles = c.out_kind == OUT_GLU || c.N >= 48 * ctx->num_sms ? 2 : 1;
-        const size_t smem = size_t(c.M) * gemv_mma_pitch(c.K) + size_t(8) * tiles * 16 * 8 * sizeof(float);
         const int ctas = (c.N + tiles * 16 - 1) / (tiles * 16);
-        return tiles == 2 ? launch_gemv(ctx, gemv_bf16_mma_kernel<2>, g, ctas, smem) : launch_gemv(ctx, gemv_bf16_mma_kernel<1>, g, ctas, smem);
+        return tiles == 2 ? launch_gemv(ctx, gemv_bf16_mma_kernel<2>, g, ctas, 0) : launch_gemv(ctx, gemv_bf16_mma_kernel<1>, g, ctas, 0);
     }
     const bool f32 = c.out_kind == OUT_F32;
     const long long out_words = f32 ? c.N : c.out_kind == OUT_GLU ? c.N / 4 : (std::min(c.N, c.tail_col) + 1) / 2;

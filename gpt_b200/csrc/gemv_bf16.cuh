@@ -140,7 +140,8 @@ gemv_bf16_kernel(const GemvParams p)
 }
 
 // Two to eight rows: the same stream of weights as the A operand of m16n8k16 products (16 weight rows, up to eight rows of x).  A
-// block takes TILES x 16 weight rows (OUT_GLU: 16 gate rows and their 16 up rows) and its eight warps share k.  The order of k inside a block
+// block takes TILES x 16 weight rows (OUT_GLU: 16 gate rows and their 16 up rows) and its eight warps share k, so no value of x is read
+// twice by a block and x comes straight from L2.  The order of k inside a block
 // of 32 is permuted alike on both sides so that a lane loads 16 contiguous bytes of a row: piece c of a block (8 values) feeds
 // two products, values 0-3 the first and 4-7 the second.
 constexpr int kGemvMmaUnroll = 4;   // blocks of 32 k in flight per warp
@@ -152,17 +153,13 @@ __device__ __forceinline__ void gemv_mma_bf16(float (&d)[4], uint32_t a0, uint32
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-__host__ __device__ inline int gemv_mma_pitch(int k) { return (k + 31) / 32 * 64 + ((k + 31) / 32 % 2 == 0 ? 64 : 0); }   // bytes, an odd multiple of 64
-
 template <int TILES>
 __global__ void __launch_bounds__(kGemvThreads)
 gemv_bf16_mma_kernel(const GemvParams p)
 {
-    extern __shared__ __align__(16) uint8_t gemv_sm[];   // x [M][pitch], then sums [8 warps][TILES * 16][8]
+    __shared__ float sums[8 * TILES * 16 * 8];   // [warp][weight row][row of x]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, c = lane & 3;
-    const int pitch = gemv_mma_pitch(p.K);
-    float *sums = reinterpret_cast<float *>(gemv_sm + p.M * pitch);
     // weight rows of the block's tiles
     int row[TILES];
 #pragma unroll
@@ -187,22 +184,18 @@ gemv_bf16_mma_kernel(const GemvParams p)
     fetch(first);
     grid_dependency_wait();
     grid_dependency_launch();
-    const int pieces = pitch / 16;
-    for (int i = threadIdx.x; i < p.M * pieces; i += kGemvThreads) {
-        const int m = i / pieces, q = i % pieces;
-        *reinterpret_cast<uint4 *>(gemv_sm + m * pitch + q * 16) = q * 8 < p.K ? *reinterpret_cast<const uint4 *>(p.x + m * p.ldx + q * 8) : make_uint4(0u, 0u, 0u, 0u);
-    }
-    __syncthreads();
     float acc[TILES][4] = {};
     const bool live = g < p.M;   // this lane's row of x
-    const uint8_t *xs = gemv_sm + (live ? g : 0) * pitch + c * 16;
+    const uint16_t *xs = p.x + (live ? g : 0) * p.ldx + c * 8;
     for (int blk = first; blk < end; blk += kGemvMmaUnroll) {
         if (blk > first) fetch(blk);
+        uint4 xv[kGemvMmaUnroll];
+#pragma unroll
+        for (int u = 0; u < kGemvMmaUnroll; ++u)
+            xv[u] = live && blk + u < end && (blk + u) * 32 + c * 8 < p.K ? *reinterpret_cast<const uint4 *>(xs + (blk + u) * 32) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
         for (int u = 0; u < kGemvMmaUnroll; ++u) {
-            if (blk + u >= end) continue;
-            uint4 x = *reinterpret_cast<const uint4 *>(xs + (blk + u) * 64);
-            if (!live) x = make_uint4(0u, 0u, 0u, 0u);
+            const uint4 x = xv[u];
 #pragma unroll
             for (int t = 0; t < TILES; ++t) {
                 const uint4 a = wv[u][t][0], b = wv[u][t][1];
