@@ -977,7 +977,7 @@ private:
     size_t fixed_state_ = 0, position_bytes_ = 0;
     std::vector<void *> weights_, work_;
     std::vector<Slot> slots_;
-    int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8, segment_tokens_ = 512;
+    int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8, segment_tokens_ = 1024;
     T *expanded_ = nullptr;
     size_t expanded_count_ = 0;
     float *scratch_ = nullptr;

@@ -353,7 +353,7 @@ int gptb200_model_step_count(gptb200_model *m);
  *   options         "pass_rows" (most rows of one pass of a step, default 4096), "expand_rows" (latent attention in bf16: shortest portion
  *                   whose keys and values are expanded for the tensor cores, default 32; shorter ones use the latents as they are),
  *                   "chunk_rows" (Mamba-2 in bf16: shortest portion that runs in chunks on the tensor cores, default 8; shorter ones token by
- *                   token), "segment_tokens" (Mamba-2 prompts: tokens per segment of the segments that run side by side, default 512) and those of gptb200_ctx_set_option */
+ *                   token), "segment_tokens" (Mamba-2 prompts: tokens per segment of the segments that run side by side, default 1024) and those of gptb200_ctx_set_option */
 typedef enum gptb200_dtype { GPTB200_DTYPE_BF16 = 0, GPTB200_DTYPE_F32 = 1 } gptb200_dtype;
 typedef struct gptb200_decoder gptb200_decoder;
 int gptb200_decoder_check_config(const char *config_json, char *message, size_t capacity);   /* host only */

@@ -99,6 +99,10 @@ def test_prompt_against_decoding_and_portions_of_many_sizes(tmp_path, dtype):
         assert dm.close(got, want, TOL[dtype]), cuts
     model.set_option("pass_rows", 70)      # the step itself works in passes
     assert dm.close(whole(model, tokens), want, TOL[dtype])
+    model.set_option("pass_rows", 4096)
+    model.set_option("segment_tokens", 64)  # segments of one chunk side by side
+    for cuts in ((1 << 20,), (130, 100, 70)):
+        assert dm.close(whole(model, tokens, cuts), want, TOL[dtype]), cuts
     model.close_model()
 
 
