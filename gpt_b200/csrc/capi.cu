@@ -738,10 +738,13 @@ int run_linear_bf16_impl(gptb200_ctx *ctx, const Bf16Linear &c)
         return fail(ctx, GPTB200_ERR_INVALID_ARG, "bf16 product: sizes or alignment (M=%d N=%d K=%d lda=%lld kind=%d)", c.M, c.N, c.K, c.lda, c.out_kind);
     if (c.M <= ctx->gemv_rows && (c.M > 1 || size_t(c.K) * 2 <= 200 * 1024)) {
         GemvParams g{c.M, c.N, c.K, static_cast<const uint16_t *>(c.a), c.lda, static_cast<const uint16_t *>(c.w), c.out_kind, c.out, c.ldo, c.tail, c.tail_col, c.tail_pitch,
-                     static_cast<const uint16_t *>(c.factor), c.factor_rows, c.factor_pitch};
+                     static_cast<const uint16_t *>(c.factor), c.factor_rows, c.factor_pitch, 1};
         if (c.M == 1) {
             const int pairs = c.out_kind == OUT_GLU ? c.N / 2 : (c.N + 1) / 2, per_cta = kGemvThreads / 32;
-            return launch_gemv(ctx, gemv_bf16_kernel, g, std::max(1, std::min((pairs + per_cta - 1) / per_cta, ctx->num_sms * 4)), size_t(c.K) * 2);
+            // few weight rows: several warps share a pair (each at least 256 of k), so that the loads of a narrow layer come from all SMs
+            while (g.k_warps < 8 && pairs * g.k_warps * 2 <= ctx->num_sms * 16 && c.K / (g.k_warps * 2) >= 256) g.k_warps *= 2;
+            const int need = (pairs * g.k_warps + per_cta - 1) / per_cta;
+            return launch_gemv(ctx, gemv_bf16_kernel, g, g.k_warps > 1 ? need : std::max(1, std::min(need, ctx->num_sms * 4)), size_t(c.K) * 2);
         }
         const int tiles = c.out_kind == OUT_GLU || c.N >= 48 * ctx->num_sms ? 2 : 1;
         const int ctas = (c.N + tiles * 16 - 1) / (tiles * 16);

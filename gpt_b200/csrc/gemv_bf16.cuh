@@ -28,6 +28,7 @@ struct GemvParams {
     const uint16_t *factor;
     const int *factor_rows;
     int factor_pitch;
+    int k_warps;            // one row: warps of a block that share a pair of weight rows (1, 2, 4, 8)
 };
 
 constexpr int kGemvThreads = 256;
@@ -85,11 +86,14 @@ static __global__ void __launch_bounds__(kGemvThreads)
 gemv_bf16_kernel(const GemvParams p)
 {
     extern __shared__ uint4 gemv_x[];   // [K / 8]
+    __shared__ float2 parts[kGemvThreads / 32];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int chunks = p.K >> 3;
     const int pairs = p.out_kind == OUT_GLU ? p.N / 2 : (p.N + 1) / 2;
-    const int stride = gridDim.x * (kGemvThreads / 32);
-    int pair = blockIdx.x * (kGemvThreads / 32) + warp;
+    const int per_block = (kGemvThreads / 32) / p.k_warps, stride = gridDim.x * per_block;
+    int pair = blockIdx.x * per_block + warp / p.k_warps;
+    // this warp's share of k, in chunks of 8
+    const int share = (chunks + p.k_warps - 1) / p.k_warps, begin = (warp % p.k_warps) * share, end = min(chunks, begin + share);
 
     uint4 wa[kGemvUnroll], wb[kGemvUnroll];
     auto fetch = [&](int i, int c0) {
@@ -100,23 +104,23 @@ gemv_bf16_kernel(const GemvParams p)
 #pragma unroll
         for (int u = 0; u < kGemvUnroll; ++u) {
             const int c = c0 + u * 32 + lane;
-            wa[u] = c < chunks ? __ldg(a + c) : make_uint4(0u, 0u, 0u, 0u);
-            wb[u] = c < chunks && rb < p.N ? __ldg(b + c) : make_uint4(0u, 0u, 0u, 0u);
+            wa[u] = c < end ? __ldg(a + c) : make_uint4(0u, 0u, 0u, 0u);
+            wb[u] = c < end && rb < p.N ? __ldg(b + c) : make_uint4(0u, 0u, 0u, 0u);
         }
     };
-    if (pair < pairs) fetch(pair, 0);
+    if (pair < pairs) fetch(pair, begin);
     grid_dependency_wait();
     grid_dependency_launch();
     for (int i = threadIdx.x; i < chunks; i += kGemvThreads) gemv_x[i] = *(reinterpret_cast<const uint4 *>(p.x) + i);
     __syncthreads();
     for (; pair < pairs; pair += stride) {
         float sa = 0.0f, sb = 0.0f;
-        for (int c0 = 0; c0 < chunks; c0 += 32 * kGemvUnroll) {
-            if (c0 > 0) fetch(pair, c0);
+        for (int c0 = begin; c0 < end; c0 += 32 * kGemvUnroll) {
+            if (c0 > begin) fetch(pair, c0);
 #pragma unroll
             for (int u = 0; u < kGemvUnroll; ++u) {
                 const int c = c0 + u * 32 + lane;
-                if (c < chunks) {
+                if (c < end) {
                     const uint4 xv = gemv_x[c];
                     sa = dot8(wa[u], xv, sa);
                     sb = dot8(wb[u], xv, sb);
@@ -124,7 +128,7 @@ gemv_bf16_kernel(const GemvParams p)
             }
         }
         const int done = pair;
-        if (pair + stride < pairs) fetch(pair + stride, 0);   // the next pair's first weights travel during the reduction
+        if (pair + stride < pairs) fetch(pair + stride, begin);   // the next pair's first weights travel during the reduction
         int ra, rb;
         gemv_pair(done, p.out_kind, ra, rb);
 #pragma unroll
@@ -132,7 +136,26 @@ gemv_bf16_kernel(const GemvParams p)
             sa += __shfl_xor_sync(0xffffffffu, sa, o);
             sb += __shfl_xor_sync(0xffffffffu, sb, o);
         }
+        if (p.k_warps > 1) {
+            if (lane == 0) parts[warp] = make_float2(sa, sb);
+            continue;   // the launch gives every warp at most one pair then
+        }
         if (lane == 0) {
+            gemv_emit(p, 0, ra, sa, sb);
+            if (p.out_kind != OUT_GLU && rb < p.N) gemv_emit(p, 0, rb, sb, 0.0f);
+        }
+    }
+    if (p.k_warps > 1) {
+        __syncthreads();
+        const int done = blockIdx.x * per_block + static_cast<int>(threadIdx.x);
+        if (static_cast<int>(threadIdx.x) < per_block && done < pairs) {
+            float sa = 0.0f, sb = 0.0f;
+            for (int i = 0; i < p.k_warps; ++i) {
+                sa += parts[threadIdx.x * p.k_warps + i].x;
+                sb += parts[threadIdx.x * p.k_warps + i].y;
+            }
+            int ra, rb;
+            gemv_pair(done, p.out_kind, ra, rb);
             gemv_emit(p, 0, ra, sa, sb);
             if (p.out_kind != OUT_GLU && rb < p.N) gemv_emit(p, 0, rb, sb, 0.0f);
         }

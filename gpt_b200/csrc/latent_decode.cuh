@@ -307,7 +307,7 @@ latent_combine_kernel(__nv_bfloat16 *__restrict__ out, int ld_out, const float *
     const float *po = part_o + (static_cast<long long>(blockIdx.y) * s.heads + h) * splits * s.rank_pitch;
     for (int j = tid; j < s.rank_pitch; j += blockDim.x) {
         float v = 0.0f;
-#pragma unroll 4
+#pragma unroll 8
         for (int i = 0; i < used; ++i) v = fmaf(po[static_cast<long long>(i) * s.rank_pitch + j], weight[i], v);
         latent[j] = v / total;
     }

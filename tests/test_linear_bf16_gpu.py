@@ -7,7 +7,7 @@ import torch
 pytestmark = pytest.mark.gpu
 
 # rows x columns x k: single rows, the weight-streaming kernel's limits, one-CTA tiles, split k, CTA pairs (whole tiles and cut ranges)
-SHAPES = [(1, 64, 64), (3, 320, 72), (8, 1088, 4096), (9, 64, 8), (17, 192, 200), (100, 576, 1032), (129, 64, 64), (300, 1536, 768), (1000, 320, 512), (2048, 2048, 1024),
+SHAPES = [(1, 64, 64), (1, 768, 3072), (1, 2048, 4104), (1, 4160, 1032), (3, 320, 72), (8, 1088, 4096), (9, 64, 8), (17, 192, 200), (100, 576, 1032), (129, 64, 64), (300, 1536, 768), (1000, 320, 512), (2048, 2048, 1024),
           (2500, 2944, 2048), (257, 4096, 4096)]
 
 
