@@ -744,7 +744,8 @@ int run_linear_bf16_impl(gptb200_ctx *ctx, const Bf16Linear &c)
             // few weight rows: several warps share a pair (each at least 256 of k), so that the loads of a narrow layer come from all SMs
             while (g.k_warps < 8 && pairs * g.k_warps * 2 <= ctx->num_sms * 16 && c.K / (g.k_warps * 2) >= 256) g.k_warps *= 2;
             const int need = (pairs * g.k_warps + per_cta - 1) / per_cta;
-            return launch_gemv(ctx, gemv_bf16_kernel, g, g.k_warps > 1 ? need : std::max(1, std::min(need, ctx->num_sms * 4)), size_t(c.K) * 2);
+            return g.k_warps > 1 ? launch_gemv(ctx, gemv_bf16_kernel<true>, g, need, size_t(c.K) * 2)
+                                 : launch_gemv(ctx, gemv_bf16_kernel<false>, g, std::max(1, std::min(need, ctx->num_sms * 4)), size_t(c.K) * 2);
         }
         const int tiles = c.out_kind == OUT_GLU || c.N >= 48 * ctx->num_sms ? 2 : 1;
         const int ctas = (c.N + tiles * 16 - 1) / (tiles * 16);

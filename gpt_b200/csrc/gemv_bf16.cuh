@@ -82,18 +82,21 @@ __device__ __forceinline__ void gemv_pair(int i, int out_kind, int &ra, int &rb)
     }
 }
 
-static __global__ void __launch_bounds__(kGemvThreads)
+// SHARED: p.k_warps warps share a pair of weight rows and every warp has at most one pair.
+template <bool SHARED>
+__global__ void __launch_bounds__(kGemvThreads)
 gemv_bf16_kernel(const GemvParams p)
 {
     extern __shared__ uint4 gemv_x[];   // [K / 8]
-    __shared__ float2 parts[kGemvThreads / 32];
+    __shared__ float2 parts[SHARED ? kGemvThreads / 32 : 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int chunks = p.K >> 3;
     const int pairs = p.out_kind == OUT_GLU ? p.N / 2 : (p.N + 1) / 2;
-    const int per_block = (kGemvThreads / 32) / p.k_warps, stride = gridDim.x * per_block;
-    int pair = blockIdx.x * per_block + warp / p.k_warps;
+    const int k_warps = SHARED ? p.k_warps : 1;
+    const int per_block = (kGemvThreads / 32) / k_warps, stride = gridDim.x * per_block;
+    int pair = blockIdx.x * per_block + warp / k_warps;
     // this warp's share of k, in chunks of 8
-    const int share = (chunks + p.k_warps - 1) / p.k_warps, begin = (warp % p.k_warps) * share, end = min(chunks, begin + share);
+    const int share = (chunks + k_warps - 1) / k_warps, begin = SHARED ? (warp % k_warps) * share : 0, end = SHARED ? min(chunks, begin + share) : chunks;
 
     uint4 wa[kGemvUnroll], wb[kGemvUnroll];
     auto fetch = [&](int i, int c0) {
@@ -136,23 +139,23 @@ gemv_bf16_kernel(const GemvParams p)
             sa += __shfl_xor_sync(0xffffffffu, sa, o);
             sb += __shfl_xor_sync(0xffffffffu, sb, o);
         }
-        if (p.k_warps > 1) {
+        if (SHARED) {
             if (lane == 0) parts[warp] = make_float2(sa, sb);
-            continue;   // the launch gives every warp at most one pair then
+            continue;
         }
         if (lane == 0) {
             gemv_emit(p, 0, ra, sa, sb);
             if (p.out_kind != OUT_GLU && rb < p.N) gemv_emit(p, 0, rb, sb, 0.0f);
         }
     }
-    if (p.k_warps > 1) {
+    if (SHARED) {
         __syncthreads();
         const int done = blockIdx.x * per_block + static_cast<int>(threadIdx.x);
         if (static_cast<int>(threadIdx.x) < per_block && done < pairs) {
             float sa = 0.0f, sb = 0.0f;
-            for (int i = 0; i < p.k_warps; ++i) {
-                sa += parts[threadIdx.x * p.k_warps + i].x;
-                sb += parts[threadIdx.x * p.k_warps + i].y;
+            for (int i = 0; i < k_warps; ++i) {
+                sa += parts[threadIdx.x * k_warps + i].x;
+                sb += parts[threadIdx.x * k_warps + i].y;
             }
             int ra, rb;
             gemv_pair(done, p.out_kind, ra, rb);
