@@ -106,6 +106,22 @@ def test_prompt_against_decoding_and_portions_of_many_sizes(tmp_path, dtype):
     model.close_model()
 
 
+@pytest.mark.parametrize("layers", [
+    [dm.latent(heads=2, dim=128, rot_dim=64, vdim=128, kv_rank=96)], [dm.latent(heads=1, dim=192, rot_dim=64, vdim=80, kv_rank=520)], [dm.latent(heads=2, dim=48, vdim=136, kv_rank=72)],
+    [dm.latent(heads=18, dim=8, rot_dim=8, vdim=8, kv_rank=24)], [dm.mamba(heads=2, vdim=64, state=128, groups=1, norm_groups=1), dm.mamba(heads=2, vdim=40, state=136, groups=2, norm_groups=1)],
+], ids=["deep heads", "one stage", "wide values", "many heads", "large states"])
+def test_large_heads_and_states(tmp_path, layers):
+    """Sizes that take other rings, fragments and fallbacks of the kernels, over several key blocks and chunks."""
+    c, w = build(layers, {}, {}, 24)   # weights without rows that bf16 rounding alone moves far (single heads that nearly cancel before a norm)
+    tokens = np.random.default_rng(22).integers(0, c["vocab"], 330)
+    want = budurax.forward(c, w, tokens)
+    for dtype in DTYPES:
+        model = load(tmp_path, c, w, dtype)
+        for cuts in ((1 << 20,), (200, 33, 90, 5, 1)):
+            assert dm.close(whole(model, tokens, cuts), want, TOL[dtype]), (dtype, cuts)
+        model.close_model()
+
+
 def test_long_decoding(tmp_path):
     c, w = build(MIXED["layers"], {}, {}, 4)
     tokens = np.random.default_rng(9).integers(0, c["vocab"], 700)
