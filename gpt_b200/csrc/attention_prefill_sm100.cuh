@@ -1,4 +1,5 @@
-// Latent attention over expanded keys and values on the tensor cores (prompts and portions of prompts of one request).
+// Causal attention over key and value matrices on the tensor cores (prompts and portions of prompts of one request): latent attention over
+// expanded keys and values, grouped attention over its cache.
 //
 // One CTA takes one head and 256 query rows as two tiles of 128; per block of 128 keys
 //   S = Q K^T       tcgen05.mma, Q and K from shared memory (unrotated and rotated parts as separate 64-column blocks), S in TMEM
@@ -15,7 +16,7 @@
 // Every wait is bounded, as in the GEMM kernels.
 #pragma once
 
-#include "latent_attention.cuh"
+#include "decoder_rows.cuh"
 
 namespace gptb200 {
 namespace dec {
@@ -23,13 +24,15 @@ namespace dec {
 struct PrefillParams {
     int rows, pos0;            // the request's rows of this step and the position of the first
     int heads, vdim, v_pad;    // v_pad: value columns per head, a multiple of 16, at most 128
-    int q_stride, q_rot;       // words-aligned columns: per head, start of the rotated part
-    int dim_pad, rot_pad;      // multiples of 16
+    int kv_share;              // query heads per key / value head
+    int q_stride, q_rot;       // words-aligned columns: per head, start of the part whose keys all heads share
+    int dim_pad, rot_pad;      // multiples of 16; rot_pad: width of that part (0: none)
     int u_blocks, r_blocks, v_blocks;   // 64-column blocks of the three parts
     int k_stages, v_stages;
-    int v_col0;                // first value column of head 0 in the expanded rows
-    int rot_col0;              // rotated key part in the cached rows
+    int v_col0;                // first value column of head 0 in the rows of keys and values
+    int rot_col0;              // shared key part in its rows
     float scale_log2;          // scale * log2(e)
+    float cap_log2, cap_in;    // CAPPED: cap * log2(e), 2 * scale / cap * log2(e)
     __nv_bfloat16 *out;        // [rows][ld_out], head h at h * vdim
     int ld_out;
     const __nv_bfloat16 *gate; // [rows][ld_gate], head h at h * vdim
@@ -83,10 +86,20 @@ __device__ __forceinline__ float exp2_approx(float x)
     return y;
 }
 
+__device__ __forceinline__ float rcp_approx(float x)
+{
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 }  // namespace ptx_attn
 
+// map_kv: rows of [keys of all heads | values of all heads]; map_shared: rows with the key part that all heads share.
+// CAPPED: scores become cap * tanh(score / cap), in the form cap - 2 cap / (1 + exp(2 score / cap)).
+template <bool CAPPED>
 __global__ void __launch_bounds__(kPrefillThreads, 1)
-latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_cache, const PrefillParams p)
+attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_shared, const PrefillParams p)
 {
     extern __shared__ uint8_t smem_raw[];
     const uint32_t base = (ptx::smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -109,7 +122,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     volatile uint32_t *abort_flag = tmem_slot + 1;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int head = blockIdx.y;
+    const int head = blockIdx.y, kv_head = head / p.kv_share;
     const int row_base = (gridDim.x - 1 - blockIdx.x) * 256;   // the longest rows first
     // key blocks of the two tiles
     int n_blocks[2];
@@ -138,7 +151,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         ptx::fence_mbar_init();
         ptx::prefetch_tensormap(&map_q);
         ptx::prefetch_tensormap(&map_kv);
-        ptx::prefetch_tensormap(&map_cache);
+        ptx::prefetch_tensormap(&map_shared);
     }
     if (warp == 1) {
         ptx::tmem_alloc(ptx::smem_u32(tmem_slot), 512);
@@ -170,12 +183,12 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 if (!bounded_wait(k_empty(ks), ((j / p.k_stages) & 1) ^ 1, abort_flag, p.status, DEV_TIMEOUT_PRODUCER)) { ok = false; break; }
                 ptx::mbar_arrive_expect_tx(k_full(ks), qk_blocks * kPrefillBlock);
                 const uint32_t kd = k_base + ks * qk_blocks * kPrefillBlock;
-                for (int b = 0; b < p.u_blocks; ++b) ptx::tma_load_2d(kd + b * kPrefillBlock, &map_kv, head * p.dim_pad / 2 + b * 32, j * 128, k_full(ks));
-                for (int b = 0; b < p.r_blocks; ++b) ptx::tma_load_2d(kd + (p.u_blocks + b) * kPrefillBlock, &map_cache, p.rot_col0 / 2 + b * 32, j * 128, k_full(ks));
+                for (int b = 0; b < p.u_blocks; ++b) ptx::tma_load_2d(kd + b * kPrefillBlock, &map_kv, kv_head * p.dim_pad / 2 + b * 32, j * 128, k_full(ks));
+                for (int b = 0; b < p.r_blocks; ++b) ptx::tma_load_2d(kd + (p.u_blocks + b) * kPrefillBlock, &map_shared, p.rot_col0 / 2 + b * 32, j * 128, k_full(ks));
                 if (!bounded_wait(v_empty(vs), ((j / p.v_stages) & 1) ^ 1, abort_flag, p.status, DEV_TIMEOUT_PRODUCER)) { ok = false; break; }
                 ptx::mbar_arrive_expect_tx(v_full(vs), p.v_blocks * kPrefillBlock);
                 const uint32_t vd = v_base + vs * p.v_blocks * kPrefillBlock;
-                for (int b = 0; b < p.v_blocks; ++b) ptx::tma_load_2d(vd + b * kPrefillBlock, &map_kv, (p.v_col0 + head * p.v_pad) / 2 + b * 32, j * 128, v_full(vs));
+                for (int b = 0; b < p.v_blocks; ++b) ptx::tma_load_2d(vd + b * kPrefillBlock, &map_kv, (p.v_col0 + kv_head * p.v_pad) / 2 + b * 32, j * 128, v_full(vs));
             }
         } else if (warp == 1 && lane == 0) {
             constexpr uint32_t idesc_s = ptx::make_idesc_bf16(128, 128, false, false);
@@ -254,7 +267,10 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 ptx::tmem_ld_32x32(s_addr + 32 * c, r);
                 ptx::tmem_ld_wait();
 #pragma unroll
-                for (int i = 0; i < 32; ++i) s[32 * c + i] = __uint_as_float(r[i]) * p.scale_log2;
+                for (int i = 0; i < 32; ++i) {
+                    const float x = __uint_as_float(r[i]);
+                    s[32 * c + i] = CAPPED ? fmaf(-2.0f * p.cap_log2, ptx_attn::rcp_approx(1.0f + ptx_attn::exp2_approx(x * p.cap_in)), p.cap_log2) : x * p.scale_log2;
+                }
             }
             if (j * 128 + 127 > p.pos0 + row_base + g * 128) {   // the tile's first row does not see all of this block
 #pragma unroll

@@ -708,7 +708,7 @@ int make_word_tmap(gptb200_ctx *ctx, CUtensorMap *map, const void *base, long lo
 }
 
 // Launch of a weight-streaming kernel, early when the context allows it (see the kernels' header).
-int launch_gemv(gptb200_ctx *ctx, void (*kernel)(GemvParams), const GemvParams &g, int ctas, size_t smem)
+int launch_gemv(gptb200_ctx *ctx, void (*kernel)(GemvParams), const GemvParams &g, int ctas, int groups, size_t smem)
 {
     const void *key = reinterpret_cast<const void *>(kernel);
     if (smem > 48 * 1024 && !ctx->configured.count(key)) {
@@ -716,7 +716,7 @@ int launch_gemv(gptb200_ctx *ctx, void (*kernel)(GemvParams), const GemvParams &
         ctx->configured.insert(key);
     }
     cudaLaunchConfig_t cfg{};
-    cfg.gridDim = dim3(ctas);
+    cfg.gridDim = dim3(ctas, groups);
     cfg.blockDim = dim3(kGemvThreads);
     cfg.dynamicSmemBytes = smem;
     cfg.stream = ctx->stream;
@@ -733,31 +733,32 @@ int launch_gemv(gptb200_ctx *ctx, void (*kernel)(GemvParams), const GemvParams &
 int run_linear_bf16_impl(gptb200_ctx *ctx, const Bf16Linear &c)
 {
     if (c.M <= 0 || c.N <= 0) return GPTB200_OK;
-    if (c.K <= 0 || c.K % 8 || c.lda % 8 || !aligned16(c.a) || !aligned16(c.w) || !aligned16(c.out) || (c.out_kind == OUT_GLU && c.N % 64) ||
+    if (c.K <= 0 || c.K % 8 || c.lda % 8 || !aligned16(c.a) || !aligned16(c.w) || !aligned16(c.out) || (is_glu(c.out_kind) && c.N % 64) || c.silu_cols % 32 || (c.group_cols && (c.group_cols % 256 || is_glu(c.out_kind))) ||
         (c.out_kind == OUT_BF16 && c.tail_col % 32 && c.tail_col < c.N) || (c.out_kind == OUT_GELU_MUL && (c.N % 8 || c.factor_pitch % 8 || !aligned16(c.factor))))
         return fail(ctx, GPTB200_ERR_INVALID_ARG, "bf16 product: sizes or alignment (M=%d N=%d K=%d lda=%lld kind=%d)", c.M, c.N, c.K, c.lda, c.out_kind);
     if (c.M <= ctx->gemv_rows && (c.M > 1 || size_t(c.K) * 2 <= 200 * 1024)) {
         GemvParams g{c.M, c.N, c.K, static_cast<const uint16_t *>(c.a), c.lda, static_cast<const uint16_t *>(c.w), c.out_kind, c.out, c.ldo, c.tail, c.tail_col, c.tail_pitch,
-                     static_cast<const uint16_t *>(c.factor), c.factor_rows, c.factor_pitch, 1};
+                     static_cast<const uint16_t *>(c.factor), c.factor_rows, c.factor_pitch, c.bias, c.silu_cols, c.group_cols ? c.group_cols : c.N, static_cast<long long>(c.group_rows) * c.lda, 1};
+        const int groups = (c.N + g.group_cols - 1) / g.group_cols, widest = std::min(c.N, g.group_cols);
         if (c.M == 1) {
-            const int pairs = c.out_kind == OUT_GLU ? c.N / 2 : (c.N + 1) / 2, per_cta = kGemvThreads / 32;
+            const int pairs = is_glu(c.out_kind) ? c.N / 2 : (widest + 1) / 2, per_cta = kGemvThreads / 32;
             // few weight rows: several warps share a pair (each at least 256 of k), so that the loads of a narrow layer come from all SMs
-            while (g.k_warps < 8 && pairs * g.k_warps * 2 <= ctx->num_sms * 16 && c.K / (g.k_warps * 2) >= 256) g.k_warps *= 2;
+            while (g.k_warps < 8 && groups * pairs * g.k_warps * 2 <= ctx->num_sms * 16 && c.K / (g.k_warps * 2) >= 256) g.k_warps *= 2;
             const int need = (pairs * g.k_warps + per_cta - 1) / per_cta;
-            return g.k_warps > 1 ? launch_gemv(ctx, gemv_bf16_kernel<true>, g, need, size_t(c.K) * 2)
-                                 : launch_gemv(ctx, gemv_bf16_kernel<false>, g, std::max(1, std::min(need, ctx->num_sms * 4)), size_t(c.K) * 2);
+            return g.k_warps > 1 ? launch_gemv(ctx, gemv_bf16_kernel<true>, g, need, groups, size_t(c.K) * 2)
+                                 : launch_gemv(ctx, gemv_bf16_kernel<false>, g, std::max(1, std::min(need, ctx->num_sms * 4 / groups)), groups, size_t(c.K) * 2);
         }
-        const int tiles = c.out_kind == OUT_GLU || c.N >= 48 * ctx->num_sms ? 2 : 1;
-        const int ctas = (c.N + tiles * 16 - 1) / (tiles * 16);
-        return tiles == 2 ? launch_gemv(ctx, gemv_bf16_mma_kernel<2>, g, ctas, 0) : launch_gemv(ctx, gemv_bf16_mma_kernel<1>, g, ctas, 0);
+        const int tiles = is_glu(c.out_kind) || c.N >= 48 * ctx->num_sms ? 2 : 1;
+        const int ctas = (widest + tiles * 16 - 1) / (tiles * 16);
+        return tiles == 2 ? launch_gemv(ctx, gemv_bf16_mma_kernel<2>, g, ctas, groups, 0) : launch_gemv(ctx, gemv_bf16_mma_kernel<1>, g, ctas, groups, 0);
     }
     const bool f32 = c.out_kind == OUT_F32;
-    const long long out_words = f32 ? c.N : c.out_kind == OUT_GLU ? c.N / 4 : (std::min(c.N, c.tail_col) + 1) / 2;
+    const long long out_words = f32 ? c.N : is_glu(c.out_kind) ? c.N / 4 : (std::min(c.N, c.tail_col) + 1) / 2;
     const long long ldo_words = f32 ? c.ldo : c.ldo / 2;
     if (ldo_words % 4 || c.ldo % 2) return fail(ctx, GPTB200_ERR_INVALID_ARG, "bf16 product: output pitch %lld", c.ldo);
     GemmPlanInput in{};
     in.M = c.M; in.N = (c.N + 3) & ~3; in.K = c.K / 2;      // in 4-byte words: a k-block of 32 words is 64 bf16
-    in.has_epilogue = !f32 || c.ldo != c.N || c.N % 4 != 0;   // split-K adds contiguous fp32 partial sums
+    in.has_epilogue = !f32 || c.bias || c.ldo != c.N || c.N % 4 != 0;   // split-K adds contiguous fp32 partial sums
     in.aligned = true;
     in.num_sms = ctx->max_sms > 0 ? std::min(ctx->max_sms, ctx->num_sms) : ctx->num_sms;
     in.opt_tile_n = ctx->tile_n; in.opt_max_splits = ctx->max_splits; in.opt_pair = ctx->pair; in.opt_stream_k = ctx->stream_k;
@@ -773,6 +774,8 @@ int run_linear_bf16_impl(gptb200_ctx *ctx, const Bf16Linear &c)
     p.out_kind = c.out_kind;
     p.tail = c.tail; p.tail_col = c.tail_col; p.tail_pitch = c.tail_pitch;
     p.factor = c.factor; p.factor_rows = c.factor_rows; p.factor_pitch = c.factor_pitch;
+    p.bias = c.bias; p.silu_cols = c.silu_cols;
+    p.a_group_cols = c.group_cols; p.a_group_rows = c.group_rows;
     p.epi_mode = EPI_STORE;
     float *out_base = static_cast<float *>(c.out);
     if (pair) {
@@ -792,7 +795,8 @@ int run_linear_bf16_impl(gptb200_ctx *ctx, const Bf16Linear &c)
         p.epi_mode = EPI_PARTIAL;
     }
     CUtensorMap ta, tb, to;
-    int rc = make_word_tmap(ctx, &ta, c.a, c.M, c.K / 2, c.lda / 2, kBK, kBM, false);
+    const long long a_rows = c.group_cols ? (c.N + c.group_cols - 1LL) / c.group_cols * c.group_rows : c.M;
+    int rc = make_word_tmap(ctx, &ta, c.a, a_rows, c.K / 2, c.lda / 2, kBK, kBM, false);
     if (rc == GPTB200_OK) rc = make_word_tmap(ctx, &tb, c.w, c.N, c.K / 2, c.K / 2, kBK, pair ? pl.tile_n / 2 : pl.tile_n, false);
     if (rc == GPTB200_OK && pl.splits > 1) rc = make_out_tmap(ctx, &to, out_base, pl.splits, c.M, c.N);
     if (rc == GPTB200_OK && pl.splits <= 1) rc = make_word_tmap(ctx, &to, c.out, c.M, out_words, ldo_words, f32 ? 32 : 16, 32, true);
@@ -842,9 +846,9 @@ int bf16_operand_map(gptb200_ctx *ctx, CUtensorMap *map, const void *base, long 
     return make_word_tmap(ctx, map, base, rows, cols / 2, pitch / 2, kBK, box_rows, false);
 }
 
-int run_linear_f32(gptb200_ctx *ctx, float *out, const float *a, const float *w, int M, int N, int K)
+int run_linear_f32(gptb200_ctx *ctx, float *out, const float *a, const float *w, int M, int N, int K, const float *bias)
 {
-    GemmCall c{M, N, K, a, false, w, false, out, nullptr, nullptr, false};
+    GemmCall c{M, N, K, a, false, w, false, out, nullptr, bias, false};
     c.fma_only = true;
     return run_gemm(ctx, c);
 }
@@ -1317,7 +1321,7 @@ int gptb200_memcpy_d2h(gptb200_ctx *ctx, void *dst, const void *src, size_t byte
 int gptb200_linear_bf16(gptb200_ctx *ctx, int kind, void *out, long long out_pitch, const void *x, long long x_pitch, const void *w, int m, int n, int k, float *tail,
                         int tail_col, int tail_pitch, const void *factor, const int *factor_rows, int factor_pitch)
 {
-    if (!ctx || kind < OUT_F32 || kind > OUT_GELU_MUL || m < 0 || n < 0 || k < 0) return GPTB200_ERR_INVALID_ARG;
+    if (!ctx || kind < OUT_F32 || kind > OUT_GLU_SILU || m < 0 || n < 0 || k < 0) return GPTB200_ERR_INVALID_ARG;
     if (m == 0 || n == 0) return GPTB200_OK;
     if (!out || !x || !w || (kind == OUT_BF16 && tail_col < n && !tail) || (kind == OUT_GELU_MUL && (!factor || !factor_rows)))
         return fail(ctx, GPTB200_ERR_INVALID_ARG, "null tensor pointer");

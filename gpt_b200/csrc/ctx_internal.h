@@ -138,6 +138,10 @@ struct Bf16Linear {
     const void *factor = nullptr;   // OUT_GELU_MUL
     const int *factor_rows = nullptr;
     int factor_pitch = 0;
+    const float *bias = nullptr;    // [N], added to the product
+    int silu_cols = 0;              // OUT_BF16: silu is applied to the columns before this one (a multiple of 32)
+    int group_cols = 0;             // columns [g * group_cols, (g + 1) * group_cols) multiply rows from g * group_rows on of a; 0: one group,
+    int group_rows = 0;             //   else a multiple of 256 (not with the gated kinds)
 };
 int run_linear_bf16(gptb200_ctx *ctx, const Bf16Linear &c);
 
@@ -146,7 +150,7 @@ int run_linear_bf16(gptb200_ctx *ctx, const Bf16Linear &c);
 int bf16_operand_map(gptb200_ctx *ctx, CUtensorMap *map, const void *base, long long rows, long long cols, long long pitch, int box_rows);
 
 // out[m][n] = a[m][k] . w[n][k] in fp32 FMAs only (no tensor core), whatever the context's mode.
-int run_linear_f32(gptb200_ctx *ctx, float *out, const float *a, const float *w, int M, int N, int K);
+int run_linear_f32(gptb200_ctx *ctx, float *out, const float *a, const float *w, int M, int N, int K, const float *bias = nullptr);
 
 // Grows the context's scratch buffer to at least `bytes` (waits for queued work before replacing it).
 int ensure_workspace(gptb200_ctx *ctx, size_t bytes);

@@ -9,7 +9,8 @@
 
 namespace gptb200 {
 
-// Rotary positions: pairs (i, i + dims / 2), frequency base^(-2 i / dims), optionally stretched (YaRN).
+// Rotary positions: frequency base^(-2 i / dims) of pair i, optionally stretched (YaRN).  Which dimensions form a pair -- (i, i + dims / 2)
+// or (2 i, 2 i + 1) -- is fixed by the layer kind.
 struct RotaryConfig {
     int dims = 0;
     double base = 0.0;
@@ -53,26 +54,60 @@ struct LatentConfig {
     RotaryConfig rot;
 };
 
-enum class MixerKind { Mamba2, Latent };
+// Softmax attention with grouped key / value heads, biased projections, rotated neighbouring dimensions and a sigmoid output gate.
+struct GroupedConfig {
+    int heads, kv_heads, dim, vdim;
+    double scale;
+    double softcap = 0.0;   // scores become softcap * tanh(score / softcap); 0: they stay
+    bool value_mix = false; // values are blended with those of the first layer that says so
+    bool first_values = false;   // this is that layer
+    RotaryConfig rot;
+};
+
+// Linear attention with one constant decay per head (S <- decay S + k v^T, read after the update).
+struct LightningConfig {
+    int heads, dim, vdim;
+    std::vector<double> decay;
+};
+
+// Linear attention with a decay per key channel and token and a bonus for the current token (read before the update).
+struct WkvConfig {
+    int heads, dim;
+};
+
+enum class MixerKind { Mamba2, Latent, Grouped, Lightning, Wkv };
 
 struct LayerConfig {
     MixerKind kind;
     Mamba2Config mamba{};
     LatentConfig latent{};
+    GroupedConfig grouped{};
+    LightningConfig lightning{};
+    WkvConfig wkv{};
     int ff = 0;   // width of the gated feed-forward, 0: none
 };
 
-// What an architecture fixes.  All of them: layer norms with bias before and after each sublayer, gated GELU feed-forwards.
+// How the residual stream is normed around the sublayers.
+enum class NormScheme {
+    LayerNormAround,   // layer norms with bias before and after each sublayer: x += norm(sublayer(norm(x)))
+    RmsBefore,         // root-mean-square norm, weight stored as its distance from one: x += residual_mult * sublayer(norm(x))
+};
+
+// What an architecture fixes.  All of them: gated feed-forwards.
 struct ArchitectureTraits {
     const char *name;
+    NormScheme norms;
     bool token_shift;     // the mixer input is blended with the previous token's
     bool depth_average;   // weighted sum over the results of all earlier layers after each layer
     bool token_side;      // gated per-layer token embedding after the feed-forward
+    bool silu_gate;       // feed-forward gates: silu (GELU otherwise)
+    bool pair_embedding;  // embedding times a constant, plus a row for the hashed pair (previous token, token)
 };
 
 inline const std::vector<ArchitectureTraits> &known_architectures()
 {
-    static const std::vector<ArchitectureTraits> known = {{"Budurax", true, true, true}};
+    static const std::vector<ArchitectureTraits> known = {{"Budurax", NormScheme::LayerNormAround, true, true, true, false, false},
+                                                          {"Lutelorn", NormScheme::RmsBefore, false, false, false, true, true}};
     return known;
 }
 
@@ -80,6 +115,8 @@ struct DecoderConfig {
     ArchitectureTraits traits{};
     int vocab = 0, width = 0, side_dim = 0;
     double eps = 0.0;
+    double residual_mult = 1.0, embed_scale = 1.0;
+    long long pair_buckets = 0, pair_mul_previous = 0, pair_mul_current = 0;   // buckets 0: no pair embedding
     std::vector<LayerConfig> layers;
 
     static DecoderConfig parse(const std::string &text)
@@ -98,11 +135,22 @@ struct DecoderConfig {
         c.width = j.size("width");
         c.eps = j.at("norm").num("eps");
         if (c.traits.token_side) c.side_dim = j.at("token_side").size("dim");
+        if (c.traits.norms == NormScheme::RmsBefore) c.residual_mult = j.num("residual_mult");
+        if (c.traits.pair_embedding) {
+            const Json &e = j.at("embedding");
+            c.embed_scale = e.num("scale");
+            if (e.has("bigram")) {
+                const Json &b = e.at("bigram");
+                c.pair_buckets = b.size("buckets");
+                c.pair_mul_previous = multiplier(b, "mul_prev");
+                c.pair_mul_current = multiplier(b, "mul_cur");
+            }
+        }
         const Json &layers = j.at("layers");
         if (layers.kind != Json::Array || layers.items.empty()) throw std::runtime_error("'layers' is not a list of layers");
         for (size_t i = 0; i < layers.items.size(); ++i) {
             try {
-                c.layers.push_back(parse_layer(layers.items[i], static_cast<int>(i), c.layers));
+                c.layers.push_back(parse_layer(layers.items[i], static_cast<int>(i), c.layers, c.traits));
             } catch (const std::exception &e) {
                 throw std::runtime_error("layer " + std::to_string(i) + ": " + e.what());
             }
@@ -111,6 +159,13 @@ struct DecoderConfig {
     }
 
 private:
+    // products with token ids stay far below 2^63
+    static long long multiplier(const Json &j, const char *key)
+    {
+        const double v = j.num(key);
+        if (!(v >= 0.0 && v <= 2147483647.0) || v != std::floor(v)) throw std::runtime_error(std::string("'") + key + "' is not a non-negative integer");
+        return static_cast<long long>(v);
+    }
     static RotaryConfig parse_rotary(const Json &j)
     {
         RotaryConfig r;
@@ -128,7 +183,7 @@ private:
         }
         return r;
     }
-    static LayerConfig parse_layer(const Json &j, int index, const std::vector<LayerConfig> &before)
+    static LayerConfig parse_layer(const Json &j, int index, const std::vector<LayerConfig> &before, const ArchitectureTraits &traits)
     {
         LayerConfig l{};
         const std::string &type = j.str("type");
@@ -158,6 +213,46 @@ private:
                 if (src.latent.kv_rank != a.kv_rank || src.latent.rot_dim != a.rot_dim || !(src.latent.rot == a.rot))
                     throw std::runtime_error("'kv_from': latent sizes or rotation differ");
             }
+        } else if (type == "attention") {
+            l.kind = MixerKind::Grouped;
+            GroupedConfig &a = l.grouped;
+            a.heads = m.size("heads");
+            a.kv_heads = m.size("kv_heads");
+            a.dim = m.size("dim");
+            a.vdim = m.size("vdim");
+            if (a.heads % a.kv_heads) throw std::runtime_error("'heads' is not a multiple of 'kv_heads'");
+            a.scale = m.num("scale");
+            if (m.has("softcap")) {
+                a.softcap = m.num("softcap");
+                if (!(a.softcap > 0.0)) throw std::runtime_error("'softcap' is not positive");
+            }
+            if (m.has("rot")) a.rot = parse_rotary(m.at("rot"));
+            if (a.rot.dims > a.dim) throw std::runtime_error("more rotated dimensions than 'dim'");
+            a.value_mix = m.has("v_mix") && m.flag("v_mix");
+            if (a.value_mix) {
+                a.first_values = true;
+                for (const LayerConfig &b : before)
+                    if (b.kind == MixerKind::Grouped && b.grouped.first_values) {
+                        a.first_values = false;
+                        if (b.grouped.kv_heads != a.kv_heads || b.grouped.vdim != a.vdim) throw std::runtime_error("'v_mix': the first such layer's values have other sizes");
+                    }
+            }
+        } else if (type == "lightning") {
+            l.kind = MixerKind::Lightning;
+            LightningConfig &a = l.lightning;
+            a.heads = m.size("heads");
+            a.dim = m.size("dim");
+            a.vdim = m.size("vdim");
+            const Json &d = m.at("decay");
+            if (d.kind != Json::Array || d.items.size() != static_cast<size_t>(a.heads)) throw std::runtime_error("'decay' is not a list with one number per head");
+            for (const Json &v : d.items) {
+                if (v.kind != Json::Number || !(v.number >= 0.0 && v.number <= 1.0)) throw std::runtime_error("'decay' is not between 0 and 1");
+                a.decay.push_back(v.number);
+            }
+        } else if (type == "wkv") {
+            l.kind = MixerKind::Wkv;
+            l.wkv = {m.size("heads"), m.size("dim")};
+            if (traits.norms != NormScheme::RmsBefore) throw std::runtime_error("'wkv' layers mix their own inputs: not with this architecture's norms");
         } else {
             throw std::runtime_error("unknown layer type '" + type + "'");
         }

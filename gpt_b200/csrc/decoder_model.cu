@@ -2,8 +2,8 @@
 // step over any mixture of requests, sampling, generation.
 //
 // A step takes, for each of its requests, the next tokens (a prompt, a portion of one, or a single token) and runs only those: what
-// came before is in the request's slot -- cached latents of the attention layers, convolution inputs and states of the
-// recurrent layers, the previous token's normed residual of every layer.  A slot belongs to one request from open to close and
+// came before is in the request's slot -- cached latents or keys and values of the attention layers, convolution inputs and states of
+// the recurrent layers, the previous token and its normed residual of the layers that look back at it.  A slot belongs to one request from open to close and
 // is zeroed when it is opened.
 //
 // T is the type of weights, activations and caches: bf16 (products on the tensor cores, or streamed weights for a few rows) or
@@ -15,15 +15,18 @@
 #include <type_traits>
 #include <vector>
 
+#include "attention_prefill_sm100.cuh"
 #include "ctx_internal.h"
 #include "decoder_config.h"
 #include "decoder_rows.cuh"
+#include "grouped_attention.cuh"
 #include "latent_attention.cuh"
 #include "latent_decode.cuh"
-#include "latent_prefill_sm100.cuh"
+#include "linear_attention.cuh"
 #include "mamba2.cuh"
 #include "mamba2_chunk.cuh"
 #include "safetensors.h"
+#include "wkv_chunk.cuh"
 
 using namespace gptb200;
 using namespace gptb200::dec;
@@ -89,13 +92,17 @@ public:
         size_t off = 0;
         const auto take = [&](size_t bytes) { const size_t at = off; off += (bytes + 255) & ~size_t(255); return at; };
         RC_TRY(matrix(file, &embed_, {{"embed", c_.vocab}}, W, c_.vocab, pitch_));
+        if (c_.pair_buckets > 0) {
+            RC_TRY(matrix(file, &pairs_, {{"bigram", static_cast<int>(c_.pair_buckets) + 1}}, W, static_cast<int>(c_.pair_buckets) + 1, pitch_));
+            previous_state_ = take(2 * sizeof(int));
+        }
         const TensorView *side = c_.traits.token_side ? &tensor(file, "side.embed", {c_.vocab, static_cast<long long>(c_.layers.size()) * c_.side_dim}) : nullptr;
         for (size_t i = 0; i < layers_.size(); ++i) {
             const LayerConfig &l = c_.layers[i];
             Layer &d = layers_[i];
             const std::string p = "l" + std::to_string(i) + ".", m = p + "mix.";
             RC_TRY(norm(file, &d.norm1, p + "norm1"));
-            RC_TRY(norm(file, &d.norm1b, p + "norm1b"));
+            if (norms_around()) RC_TRY(norm(file, &d.norm1b, p + "norm1b"));
             if (c_.traits.token_shift) {
                 RC_TRY(vector(file, &d.shift, p + "shift", W, pitch_));
                 d.shift_state = take(2 * size_t(pitch_) * sizeof(float));
@@ -104,7 +111,7 @@ public:
             if (l.kind == MixerKind::Mamba2) {
                 const Mamba2Config &a = l.mamba;
                 MambaShape &s = d.mamba;
-                s = {a.heads, a.vdim, a.state, a.groups, a.conv, a.norm_groups, a.inner(), a.conv_channels(), 0, 0};
+                s = {{a.heads, a.vdim, a.state, a.groups, a.inner(), 0}, a.conv, a.norm_groups, a.conv_channels(), 0};
                 d.proj_cols = pad_to(a.inner() + s.channels, 32);      // T columns; the step sizes follow
                 d.proj_n = d.proj_cols + pad_to(a.heads, 8);
                 const int rows = a.inner() + s.channels;
@@ -120,6 +127,12 @@ public:
                 RC_TRY(matrix(file, &d.w_o, {{m + "o", W}}, s.inner, pitch_, d.mix_out));
                 s.conv_state = take(2 * size_t(s.taps - 1) * s.channels * sizeof(T));
                 s.ssm_state = take(2 * size_t(a.heads) * a.state * a.vdim * sizeof(float));
+            } else if (l.kind == MixerKind::Grouped) {
+                RC_TRY(load_grouped(file, d, l.grouped, m));
+            } else if (l.kind == MixerKind::Lightning) {
+                RC_TRY(load_lightning(file, d, l.lightning, m, take));
+            } else if (l.kind == MixerKind::Wkv) {
+                RC_TRY(load_wkv(file, d, l.wkv, m, take));
             } else {
                 const LatentConfig &a = l.latent;
                 LatentShape &s = d.latent;
@@ -153,7 +166,7 @@ public:
             }
             if (l.ff > 0) {
                 RC_TRY(norm(file, &d.norm2, p + "norm2"));
-                RC_TRY(norm(file, &d.norm2b, p + "norm2b"));
+                if (norms_around()) RC_TRY(norm(file, &d.norm2b, p + "norm2b"));
                 d.ff = pad_to(l.ff, 32);
                 // groups of 32 gate rows | 32 up rows, so that one tile of the product holds both halves of its outputs
                 RC_TRY(matrix(file, &d.w_glu, {{p + "mlp.gate", l.ff}, {p + "mlp.up", l.ff}}, W, 2 * d.ff, pitch_,
@@ -175,6 +188,13 @@ public:
                 max_heads_ = std::max(max_heads_, d.mamba.heads);
                 max_inner_ = std::max(max_inner_, d.mamba.inner);
             }
+            if (l.kind == MixerKind::Lightning) max_inner_ = std::max(max_inner_, d.recurrent.inner);
+            if (l.kind == MixerKind::Wkv) {
+                mixes_ = kWkvMixes;
+                max_raw_ = std::max(max_raw_, pad_to(d.wkv.heads * d.wkv.dim, 8));
+                max_low_ = std::max(max_low_, 2 * d.wkv.rank_pad);
+            }
+            if (l.kind == MixerKind::Grouped && l.grouped.value_mix) first_values_cols_ = d.grouped.kv_heads * d.grouped.v_pad;
         }
         RC_TRY(norm(file, &final_norm_, "final.norm"));
         RC_TRY(matrix(file, &head_, {{"head", c_.vocab}}, W, vocab_pitch_, pitch_));
@@ -183,6 +203,12 @@ public:
             if (layers_[i].own_keys) {
                 layers_[i].latent.cache_per_position = position_bytes_;
                 position_bytes_ += size_t(layers_[i].latent.row_pitch) * sizeof(T);
+            }
+        for (Layer &d : layers_)
+            if (d.grouped.heads) {
+                d.grouped.cache_base = fixed_state_;
+                d.grouped.cache_per_position = position_bytes_;
+                position_bytes_ += size_t(d.grouped.row_pitch) * sizeof(T);
             }
         for (Layer &d : layers_)
             if (d.cache_owner >= 0) {
@@ -244,17 +270,22 @@ public:
             pass_rows_ = value;
             return GPTB200_OK;
         }
-        if (!strcmp(key, "chunk_rows")) {   // Mamba-2: shortest portion that takes the chunked tensor-core form (0x7fffffff: none)
+        if (!strcmp(key, "chunk_rows")) {   // recurrent layers: shortest portion that takes the chunked tensor-core form (0x7fffffff: none)
             if (value < 1) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "chunk_rows must be positive");
             chunk_rows_ = value;
             return GPTB200_OK;
         }
-        if (!strcmp(key, "segment_tokens")) {   // Mamba-2 prompts: tokens per segment (a multiple of 64)
+        if (!strcmp(key, "segment_tokens")) {   // Mamba-2 and lightning prompts: tokens per segment (a multiple of 64)
             if (value < kChunk || value % kChunk) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "segment_tokens must be a multiple of %d", kChunk);
             segment_tokens_ = value;
             return GPTB200_OK;
         }
-        if (!strcmp(key, "expand_rows")) {   // latent attention: shortest portion that takes the tensor-core form (0x7fffffff: none)
+        if (!strcmp(key, "wkv_segment_tokens")) {   // wkv prompts: tokens per segment (a multiple of 16)
+            if (value < kWkvChunk || value % kWkvChunk) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "wkv_segment_tokens must be a multiple of %d", kWkvChunk);
+            wkv_segment_tokens_ = value;
+            return GPTB200_OK;
+        }
+        if (!strcmp(key, "expand_rows")) {   // attention: shortest portion that takes the tensor-core form (0x7fffffff: none)
             if (value < 1) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "expand_rows must be positive");
             expand_rows_ = value;
             return GPTB200_OK;
@@ -398,6 +429,16 @@ private:
         float *taps = nullptr, *taps_t = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *a_log = nullptr, *d_skip = nullptr, *mix_norm = nullptr;
         LatentShape latent{};
         T *w_uk = nullptr, *w_uv = nullptr;
+        GroupedShape grouped{};
+        float *bias = nullptr, share = 0.0f;        // of the projections; of the first layer's values (negative: this is that layer)
+        bool value_mix = false;
+        RecurrentShape recurrent{};
+        float *decay = nullptr, *log_decay = nullptr;
+        int off_gate = 0;
+        WkvShape wkv{};
+        int group_cols = 0;
+        float *mix = nullptr, *w0 = nullptr, *bonus = nullptr;
+        T *w2 = nullptr;
         bool own_keys = false;
         int cache_owner = -1, rotary = -1;
         int ff = 0;
@@ -415,6 +456,9 @@ private:
     struct Piece { std::string name; int rows; };
     struct Rotary { RotaryConfig config; double *freq; double gain; size_t table; };
 
+    static constexpr int kWkvMixes = 5;   // r, k, v, gate, decay
+
+    bool norms_around() const { return c_.traits.norms == NormScheme::LayerNormAround; }
     bool valid(int slot) const { return slot >= 0 && slot < static_cast<int>(slots_.size()) && slots_[slot].open; }
 
     // ---- weights: host image, then one copy
@@ -475,11 +519,11 @@ private:
             for (int j = 0; j < cols; ++j) put(host.data() + size_t(i) * pitch + j, element(t, i * ld + first + j));
         return to_device(out, host);
     }
-    int vector(const SafeTensors &f, float **out, const std::string &name, int n, int padded = 0, std::vector<long long> shape = {})
+    int vector(const SafeTensors &f, float **out, const std::string &name, int n, int padded = 0, std::vector<long long> shape = {}, float offset = 0.0f)
     {
         const TensorView &t = tensor(f, name, shape.empty() ? std::vector<long long>{n} : shape);
         std::vector<float> host(std::max(n, padded), 0.0f);
-        for (int i = 0; i < n; ++i) host[i] = element(t, i);
+        for (int i = 0; i < n; ++i) host[i] = offset + element(t, i);
         return to_device(out, host);
     }
     int transposed(const SafeTensors &f, float **out, const std::string &name, int rows, int cols)
@@ -492,8 +536,120 @@ private:
     }
     int norm(const SafeTensors &f, Norm *out, const std::string &name)
     {
-        RC_TRY(vector(f, &out->w, name, c_.width, pitch_));
-        return vector(f, &out->b, name + ".b", c_.width, pitch_);
+        RC_TRY(vector(f, &out->w, name, c_.width, pitch_, {}, norms_around() ? 0.0f : 1.0f));
+        return norms_around() ? vector(f, &out->b, name + ".b", c_.width, pitch_) : GPTB200_OK;
+    }
+
+    // ---- mixers
+    int load_grouped(const SafeTensors &file, Layer &d, const GroupedConfig &a, const std::string &m)
+    {
+        GroupedShape &s = d.grouped;
+        s.heads = a.heads; s.kv_heads = a.kv_heads; s.dim = a.dim; s.vdim = a.vdim;
+        s.dim_pad = pad_to(a.dim, 16);
+        s.v_pad = pad_to(a.vdim, 16);
+        s.row_pitch = a.kv_heads * (s.dim_pad + s.v_pad);
+        s.off_k = a.heads * s.dim_pad;
+        s.off_v = s.off_k + a.kv_heads * s.dim_pad;
+        s.off_g = s.off_v + a.kv_heads * s.v_pad;
+        s.rot_half = a.rot.dims / 2;
+        s.scale = static_cast<float>(a.scale);
+        s.softcap = static_cast<float>(a.softcap);
+        if (std::max(s.dim_pad, s.v_pad) > 768) return fail(ctx_, GPTB200_ERR_TOO_LARGE, "attention: heads beyond 768");
+        const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim, ng = a.heads * a.vdim;
+        d.proj_n = d.proj_cols = pad_to(s.off_g + ng, 8);
+        const auto place = [&](int r) {
+            if (r < nq) return r / a.dim * s.dim_pad + r % a.dim;
+            if ((r -= nq) < nk) return s.off_k + r / a.dim * s.dim_pad + r % a.dim;
+            if ((r -= nk) < nv) return s.off_v + r / a.vdim * s.v_pad + r % a.vdim;
+            return s.off_g + r - nv;
+        };
+        RC_TRY(matrix(file, &d.w_in, {{m + "q", nq}, {m + "k", nk}, {m + "v", nv}, {m + "g", ng}}, c_.width, d.proj_n, pitch_, place));
+        std::vector<float> bias(d.proj_n, 0.0f);
+        int r = 0;
+        for (const Piece &p : {Piece{m + "q.b", nq}, Piece{m + "k.b", nk}, Piece{m + "v.b", nv}}) {
+            const TensorView &t = tensor(file, p.name, {p.rows});
+            for (int i = 0; i < p.rows; ++i, ++r) bias[place(r)] = element(t, i);
+        }
+        RC_TRY(to_device(&d.bias, bias));
+        d.value_mix = a.value_mix;
+        if (a.value_mix) d.share = a.first_values ? -1.0f : scalar(file, m + "vmix");
+        d.mix_out = pad_to(ng, 8);
+        RC_TRY(matrix(file, &d.w_o, {{m + "o", c_.width}}, ng, pitch_, d.mix_out));
+        if (a.rot.dims) d.rotary = rotary_index(a.rot);
+        return GPTB200_OK;
+    }
+
+    template <typename Take>
+    int load_lightning(const SafeTensors &file, Layer &d, const LightningConfig &a, const std::string &m, Take &&take)
+    {
+        const int nk = a.heads * a.dim, nv = a.heads * a.vdim;
+        RecurrentShape &s = d.recurrent;
+        s = {a.heads, a.vdim, a.dim, a.heads, nv, 0};
+        d.off_gate = pad_to(nv + 2 * nk, 32);
+        d.proj_n = d.proj_cols = d.off_gate + pad_to(nv, 8);
+        const int before_gate = nv + 2 * nk;
+        RC_TRY(matrix(file, &d.w_in, {{m + "v", nv}, {m + "k", nk}, {m + "q", nk}, {m + "g", nv}}, c_.width, d.proj_n, pitch_,
+                      [&](int r) { return r < before_gate ? r : d.off_gate + r - before_gate; }));
+        RC_TRY(vector(file, &d.mix_norm, m + "norm", nv));
+        d.mix_out = pad_to(nv, 8);
+        RC_TRY(matrix(file, &d.w_o, {{m + "o", c_.width}}, nv, pitch_, d.mix_out));
+        std::vector<float> decay, log_decay;
+        for (double x : a.decay) {
+            decay.push_back(static_cast<float>(x));
+            log_decay.push_back(static_cast<float>(std::max(std::log(x), -200.0)));   // nothing is left of a value after that
+        }
+        RC_TRY(to_device(&d.decay, decay));
+        RC_TRY(to_device(&d.log_decay, log_decay));
+        s.ssm_state = take(2 * size_t(a.heads) * a.dim * a.vdim * sizeof(float));
+        return GPTB200_OK;
+    }
+
+    template <typename Take>
+    int load_wkv(const SafeTensors &file, Layer &d, const WkvConfig &a, const std::string &m, Take &&take)
+    {
+        const int n = a.heads * a.dim, W = c_.width;
+        if (a.dim > 1024) return fail(ctx_, GPTB200_ERR_TOO_LARGE, "wkv: dim beyond 1024");
+        const TensorView &w1 = file.get(m + "w1");   // its shape gives the rank
+        if (w1.shape.size() != 2 || w1.shape[0] < 1) throw std::runtime_error("tensor '" + m + "w1' is not a matrix");
+        WkvShape &s = d.wkv;
+        s.heads = a.heads; s.dim = a.dim;
+        s.rank = static_cast<int>(w1.shape[0]);
+        s.rank_pad = pad_to(s.rank, 8);
+        d.group_cols = pad_to(n, 256);               // whole tiles: each group multiplies rows of its own
+        d.proj_cols = 4 * d.group_cols;
+        d.proj_n = d.proj_cols + s.rank_pad;
+        s.ld_low = s.rank_pad;
+        RC_TRY(matrix(file, &d.w_in, {{m + "r", n}, {m + "k", n}, {m + "v", n}, {m + "g", n}, {m + "w1", s.rank}}, W, d.proj_n, pitch_,
+                      [&](int r) { return std::min(r / n, 4) * d.group_cols + r - std::min(r / n, 4) * n; }));
+        // W2 twice side by side: it multiplies values that come as the sum of two bf16 values
+        s.w2_pitch = 2 * s.rank_pad;
+        const TensorView &w2 = tensor(file, m + "w2", {n, s.rank});
+        std::vector<T> image(size_t(pad_to(n, 8)) * s.w2_pitch, T(0.0f));
+        for (int i = 0; i < n; ++i)
+            for (int j = 0; j < s.rank; ++j) {
+                put(image.data() + size_t(i) * s.w2_pitch + j, element(w2, 1LL * i * s.rank + j));
+                put(image.data() + size_t(i) * s.w2_pitch + s.rank_pad + j, element(w2, 1LL * i * s.rank + j));
+            }
+        RC_TRY(to_device(&d.w2, image));
+        RC_TRY(vector(file, &d.w0, m + "w0", n));
+        RC_TRY(vector(file, &d.bonus, m + "u", n, 0, {a.heads, a.dim}));
+        RC_TRY(vector(file, &d.mix_norm, m + "norm", n));
+        std::vector<float> mix;
+        for (const char *name : {"r", "k", "v", "g", "w"}) {
+            const TensorView &t = tensor(file, m + "mu." + name, {W});
+            for (int i = 0; i < pitch_; ++i) mix.push_back(i < W ? element(t, i) : 0.0f);
+        }
+        RC_TRY(to_device(&d.mix, mix));
+        d.mix_out = pad_to(n, 8);
+        RC_TRY(matrix(file, &d.w_o, {{m + "o", W}}, n, pitch_, d.mix_out));
+        d.shift_state = take(2 * size_t(pitch_) * sizeof(float));
+        s.state = take(2 * size_t(n) * a.dim * sizeof(float));
+        return GPTB200_OK;
+    }
+    float scalar(const SafeTensors &f, const std::string &name) const
+    {
+        const TensorView &t = f.get(name);
+        return element(t.shape.empty() ? tensor(f, name, {}) : tensor(f, name, {1}), 0);
     }
     int rotary_index(const RotaryConfig &r)
     {
@@ -536,7 +692,7 @@ private:
         RC_TRY(work(&x_[0], R * P));
         RC_TRY(work(&x_[1], R * P));
         RC_TRY(work(&y_, R * P));
-        RC_TRY(work(&h_, R * P));
+        RC_TRY(work(&h_, R * P * std::max(mixes_, 1)));
         RC_TRY(work(&proj_, R * max_proj_));
         RC_TRY(work(&tail_, R * max_tail_));
         RC_TRY(work(&xbc_, R * max_channels_));
@@ -544,6 +700,11 @@ private:
         RC_TRY(work(&decay_, R * max_heads_));
         RC_TRY(work(&ssm_y_, R * max_inner_));
         RC_TRY(work(&act_, R * max_act_));
+        if (first_values_cols_) RC_TRY(work(&first_values_, R * first_values_cols_));
+        if (mixes_) {
+            RC_TRY(work(&low_, R * max_low_));
+            RC_TRY(work(&raw_, R * max_raw_));
+        }
         if (kF32) RC_TRY(work(&glu_, R * 2 * max_ff_));
         RC_TRY(work(&entries_, R));
         RC_TRY(work(&row_entry_, R));
@@ -619,7 +780,9 @@ private:
     {
         const void *key = reinterpret_cast<const void *>(kernel);
         if (smem > 48 * 1024 && !ctx_->configured.count(key)) {
-            CUDA_TRY(ctx_, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+            cudaFuncAttributes fixed{};
+            CUDA_TRY(ctx_, cudaFuncGetAttributes(&fixed, kernel));
+            CUDA_TRY(ctx_, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - static_cast<int>(fixed.sharedSizeBytes)));
             ctx_->configured.insert(key);
         }
         cudaLaunchConfig_t cfg{};
@@ -722,19 +885,27 @@ private:
                 RC_TRY(launch(mamba_conv_kernel<T>, dim3(conv_blocks + dt_blocks, run), dim3(128), 0, xbc_, ld_xbc, dt_, decay_, proj_, ld, dt_raw, ld_dt, d.taps, d.conv_b, d.dt_bias, d.a_log, s,
                               entries_, row_entry_, conv_blocks, row0));
             }
-            RC_TRY(k == 2 ? mamba_chunks(d, parts, entry0, n, ld_xbc) : mamba_tokens(d, entry0, n, ld_xbc));
+            RC_TRY(k == 2 ? recurrent_chunks(s, {xbc_, ld_xbc, dt_, decay_, s.heads, d.d_skip}, parts, entry0, n) : mamba_tokens(d, entry0, n, ld_xbc));
         }
         const int part = s.inner / s.norm_groups;
         return launch(mamba_gated_norm_kernel<T>, dim3(rows, s.norm_groups), dim3(std::min(256, pad_to((part + 3) / 4, 32))), size_t(part) * sizeof(float), act_, d.mix_out,
                       static_cast<const float *>(ssm_y_), static_cast<const T *>(proj_), ld, static_cast<const float *>(d.mix_norm), s, static_cast<float>(c_.eps));
     }
 
-    int mamba_chunks(const Layer &d, const std::vector<Part> &parts, int entry0, int n, int ld_xbc)
+    // Inputs of the chunked recurrence: rows of values | state inputs | state outputs (RecurrentShape), steps (null: ones), log-decays,
+    // skip (null: none).
+    struct ChunkInputs {
+        const T *rows;
+        int ld;
+        const float *steps, *log_decay;
+        int ld_decay;
+        const float *skip;
+    };
+    int recurrent_chunks(const RecurrentShape &s, const ChunkInputs &in, const std::vector<Part> &parts, int entry0, int n)
     {
         if constexpr (kF32) {
-            return mamba_tokens(d, entry0, n, ld_xbc);
+            return fail(ctx_, GPTB200_ERR_INVALID_ARG, "chunked recurrence in fp32");
         } else {
-            const MambaShape &s = d.mamba;
             // segments that run side by side when a request alone would leave most of its time to one chunk after the other
             int longest = 0;
             for (int i = 0; i < n; ++i) longest = std::max(longest, parts[entry0 + i].count);
@@ -748,11 +919,11 @@ private:
                 RC_TRY(scratch(pieces * (size_t(s.state) * s.vdim + 1)));
                 seg_state = scratch_;
                 seg_decay = scratch_ + pieces * s.state * s.vdim;
-                RC_TRY(launch(mamba_chunk_kernel<true>, dim3(blocks, n, segments - 1), dim3(kChunkThreads), smem, ssm_y_, xbc_, ld_xbc, dt_, decay_, d.d_skip, s, entries_ + entry0, tokens,
-                              segments, seg_state, seg_decay));
+                RC_TRY(launch(mamba_chunk_kernel<true>, dim3(blocks, n, segments - 1), dim3(kChunkThreads), smem, ssm_y_, in.rows, in.ld, in.steps, in.log_decay, in.ld_decay, in.skip, s,
+                              entries_ + entry0, tokens, segments, seg_state, seg_decay));
             }
-            return launch(mamba_chunk_kernel<false>, dim3(blocks, n, segments), dim3(kChunkThreads), smem, ssm_y_, xbc_, ld_xbc, dt_, decay_, d.d_skip, s, entries_ + entry0, tokens, segments,
-                          seg_state, seg_decay);
+            return launch(mamba_chunk_kernel<false>, dim3(blocks, n, segments), dim3(kChunkThreads), smem, ssm_y_, in.rows, in.ld, in.steps, in.log_decay, in.ld_decay, in.skip, s,
+                          entries_ + entry0, tokens, segments, seg_state, seg_decay);
         }
     }
 
@@ -821,10 +992,11 @@ private:
     }
 
     // Stages of the tensor-core kernel's rings; 0: its tiles do not fit (large heads), the absorbed form serves any number of rows.
-    int prefill_stages(const LatentShape &s, int *v_stages) const
+    int prefill_stages(const LatentShape &s, int *v_stages) const { return prefill_stages(s.dim_pad, s.row_pitch - s.rank_pitch, s.v_pad, v_stages); }
+    int prefill_stages(int dim_pad, int shared_pad, int v_pad, int *v_stages) const
     {
-        const int u = (s.dim_pad + 63) / 64, r = (s.row_pitch - s.rank_pitch + 63) / 64, v = (s.v_pad + 63) / 64;
-        if (s.v_pad > 128) return 0;
+        const int u = (dim_pad + 63) / 64, r = (shared_pad + 63) / 64, v = (v_pad + 63) / 64;
+        if (v_pad > 128) return 0;
         for (const auto &st : {std::pair<int, int>{3, 3}, {2, 2}, {2, 1}, {1, 1}})
             if (prefill_smem_bytes(u, r, v, st.first, st.second) <= 232448) {
                 *v_stages = st.second;
@@ -865,6 +1037,7 @@ private:
             PrefillParams p{};
             p.rows = part.count; p.pos0 = slot.length;
             p.heads = s.heads; p.vdim = s.vdim; p.v_pad = s.v_pad;
+            p.kv_share = 1;
             p.q_stride = s.q_stride; p.q_rot = s.dim_pad;
             p.dim_pad = s.dim_pad; p.rot_pad = s.row_pitch - s.rank_pitch;
             p.u_blocks = (p.dim_pad + 63) / 64; p.r_blocks = (p.rot_pad + 63) / 64; p.v_blocks = (s.v_pad + 63) / 64;
@@ -875,7 +1048,7 @@ private:
             p.out = act_ + size_t(part.row0) * d.mix_out; p.ld_out = d.mix_out;
             p.gate = q + s.off_g; p.ld_gate = d.proj_cols;
             p.status = ctx_->d_status;
-            return launch(latent_prefill_kernel, dim3((part.count + 255) / 256, s.heads), dim3(kPrefillThreads),
+            return launch(attention_prefill_kernel<false>, dim3((part.count + 255) / 256, s.heads), dim3(kPrefillThreads),
                           size_t(prefill_smem_bytes(p.u_blocks, p.r_blocks, p.v_blocks, p.k_stages, p.v_stages)), mq, mkv, mc, p);
         }
     }
@@ -918,33 +1091,317 @@ private:
                       d.own_keys ? 1 : 0, entries_, row_entry_, row0);
     }
 
-    // All kernels of one step; everything that changes from step to step is read from device memory.
-    int kernels(const std::vector<Part> &parts, int rows, int n_want)
+    // ---- grouped attention
+    int grouped(const Layer &d, const std::vector<Part> &parts, int rows)
     {
-        const float eps = static_cast<float>(c_.eps);
-        RC_TRY(launch(embed_rows_kernel<T>, dim3(rows), dim3(row_threads(rows)), 0, states_, static_cast<const T *>(embed_), static_cast<const int *>(tokens_), pitch_));
+        const GroupedShape &s = d.grouped;
+        if constexpr (kF32) {
+            RC_TRY(run_linear_f32(ctx_, proj_, h_, d.w_in, rows, d.proj_n, pitch_, d.bias));
+        } else {
+            Bf16Linear c{};
+            c.M = rows; c.N = d.proj_n; c.K = pitch_; c.a = h_; c.lda = pitch_; c.w = d.w_in; c.out_kind = OUT_BF16; c.out = proj_; c.ldo = d.proj_cols;
+            c.bias = d.bias;
+            RC_TRY(run_linear_bf16(ctx_, c));
+        }
+        const float2 *table = d.rotary >= 0 ? table_ + rotaries_[d.rotary].table : nullptr;
+        RC_TRY(launch(grouped_prepare_kernel<T>, dim3(rows), dim3(256), 0, proj_, d.proj_cols, table, d.value_mix ? first_values_ : nullptr, d.share, s, entries_, row_entry_));
+        if constexpr (kF32) {
+            const int widest = std::max(s.dim, s.v_pad);
+            const auto run = [&](auto kernel) {
+                return launch(kernel, dim3(s.heads, rows), dim3(kGroupedWarps * 32), size_t(kGroupedWarps) * s.v_pad * sizeof(float), act_, d.mix_out, static_cast<const T *>(proj_),
+                              static_cast<long long>(d.proj_cols), s, entries_, row_entry_);
+            };
+            if (widest <= 64) return run(grouped_rows_kernel<T, 2>);
+            if (widest <= 128) return run(grouped_rows_kernel<T, 4>);
+            if (widest <= 256) return run(grouped_rows_kernel<T, 8>);
+            return run(grouped_rows_kernel<T, 24>);
+        } else {
+            // long portions one by one on the tensor cores, runs of short ones together over ranges of positions
+            int v_stages = 0;
+            const int k_stages = prefill_stages(s.dim_pad, 0, s.v_pad, &v_stages);
+            const auto is_long = [&](const Part &p) { return k_stages > 0 && p.count >= expand_rows_; };
+            for (size_t i = 0, j; i < parts.size(); i = j) {
+                j = i + 1;
+                if (is_long(parts[i])) {
+                    RC_TRY(grouped_prompt(d, parts[i], k_stages, v_stages));
+                    continue;
+                }
+                int positions = 0;
+                for (j = i; j < parts.size() && !is_long(parts[j]); ++j) {
+                    const Slot &slot = slots_[parts[j].slot];
+                    positions = std::max(positions, generating_ ? slot.capacity : slot.length + parts[j].count);
+                }
+                RC_TRY(grouped_ranges(d, parts[i].row0, parts[j - 1].row0 + parts[j - 1].count - parts[i].row0, positions));
+            }
+            return GPTB200_OK;
+        }
+    }
+
+    // positions: most that any of the rows sees (an upper bound)
+    int grouped_ranges(const Layer &d, int row0, int rows, int positions)
+    {
+        if constexpr (kF32) {
+            return GPTB200_OK;
+        } else {
+            const GroupedShape &s = d.grouped;
+            const int share = s.heads / s.kv_heads, head_tiles = (share + 15) / 16, slices = (s.v_pad + kGroupedValues - 1) / kGroupedValues, groups = s.kv_heads * head_tiles * slices;
+            constexpr int turn = kGroupedWarps * kGroupedTile;
+            int splits = std::max(1, 2 * ctx_->num_sms / (rows * groups));
+            splits = std::min({splits, kGroupedMaxSplits, (positions + turn - 1) / turn});
+            const size_t o_count = size_t(rows) * s.heads * splits * s.v_pad, ml_count = size_t(rows) * s.heads * splits * 2;
+            RC_TRY(scratch(o_count + ml_count));
+            float *o = scratch_, *ml = o + o_count;
+            const int v_cols = std::min(s.v_pad, kGroupedValues);
+            int stages = 4;
+            while (stages > 2 && grouped_smem_bytes(s.dim_pad, v_cols, stages) > (stages == 4 ? 110 : 220) * 1024) --stages;
+            const auto split = [&](auto kernel) {
+                return launch(kernel, dim3(splits, groups, rows), dim3(kGroupedWarps * 32), size_t(grouped_smem_bytes(s.dim_pad, v_cols, stages)), o, ml, proj_, d.proj_cols, s, stages, head_tiles,
+                              entries_, row_entry_, row0);
+            };
+            RC_TRY(v_cols <= 64 ? split(grouped_split_kernel<8>) : split(grouped_split_kernel<16>));
+            return launch(grouped_combine_kernel, dim3(s.heads, rows), dim3(128), 0, act_, d.mix_out, o, ml, splits, proj_, d.proj_cols, s, entries_, row_entry_, row0);
+        }
+    }
+
+    int grouped_prompt(const Layer &d, const Part &part, int k_stages, int v_stages)
+    {
+        if constexpr (kF32) {
+            return GPTB200_OK;
+        } else {
+            const GroupedShape &s = d.grouped;
+            const Slot &slot = slots_[part.slot];
+            const T *cache = reinterpret_cast<const T *>(slot.base + s.cache_base + s.cache_per_position * slot.capacity), *q = proj_ + size_t(part.row0) * d.proj_cols;
+            CUtensorMap mq, mkv;
+            RC_TRY(bf16_operand_map(ctx_, &mq, q, part.count, d.proj_cols, d.proj_cols, 128));
+            RC_TRY(bf16_operand_map(ctx_, &mkv, cache, slot.length + part.count, s.row_pitch, s.row_pitch, 128));
+            PrefillParams p{};
+            p.rows = part.count; p.pos0 = slot.length;
+            p.heads = s.heads; p.vdim = s.vdim; p.v_pad = s.v_pad;
+            p.kv_share = s.heads / s.kv_heads;
+            p.q_stride = s.dim_pad; p.q_rot = s.dim_pad;
+            p.dim_pad = s.dim_pad; p.rot_pad = 0;
+            p.u_blocks = (s.dim_pad + 63) / 64; p.r_blocks = 0; p.v_blocks = (s.v_pad + 63) / 64;
+            p.k_stages = k_stages; p.v_stages = v_stages;
+            p.v_col0 = s.kv_heads * s.dim_pad;
+            constexpr double kLog2e = 1.4426950408889634;
+            p.scale_log2 = static_cast<float>(s.scale * kLog2e);
+            if (s.softcap > 0.0f) {
+                p.cap_log2 = static_cast<float>(s.softcap * kLog2e);
+                p.cap_in = static_cast<float>(2.0 * s.scale / s.softcap * kLog2e);
+            }
+            p.out = act_ + size_t(part.row0) * d.mix_out; p.ld_out = d.mix_out;
+            p.gate = q + s.off_g; p.ld_gate = d.proj_cols;
+            p.status = ctx_->d_status;
+            const size_t smem = size_t(prefill_smem_bytes(p.u_blocks, 0, p.v_blocks, k_stages, v_stages));
+            const dim3 grid((part.count + 255) / 256, s.heads);
+            return s.softcap > 0.0f ? launch(attention_prefill_kernel<true>, grid, dim3(kPrefillThreads), smem, mq, mkv, mkv, p)
+                                    : launch(attention_prefill_kernel<false>, grid, dim3(kPrefillThreads), smem, mq, mkv, mkv, p);
+        }
+    }
+
+    // ---- linear attention with constant decays
+    int lightning(const Layer &d, const std::vector<Part> &parts, int rows)
+    {
+        const RecurrentShape &s = d.recurrent;
+        if constexpr (kF32) {
+            RC_TRY(run_linear_f32(ctx_, proj_, h_, d.w_in, rows, d.proj_n, pitch_));
+            RC_TRY(launch(silu_columns_kernel, dim3(rows), dim3(256), 0, proj_, d.off_gate, d.proj_cols));
+        } else {
+            Bf16Linear c{};
+            c.M = rows; c.N = d.proj_n; c.K = pitch_; c.a = h_; c.lda = pitch_; c.w = d.w_in; c.out_kind = OUT_BF16; c.out = proj_; c.ldo = d.proj_cols;
+            c.silu_cols = d.off_gate;
+            RC_TRY(run_linear_bf16(ctx_, c));
+        }
+        RC_TRY(runs(parts, [&](const Part &p) { return !kF32 && s.state <= kChunkMaxState && p.count >= chunk_rows_; }, [&](bool chunks, int entry0, int n) {
+            if (chunks) return recurrent_chunks(s, {proj_, d.proj_cols, nullptr, d.log_decay, 0, nullptr}, parts, entry0, n);
+            const bool keep_state = lightning_smem_floats(s.state, true) * sizeof(float) <= 96 * 1024;
+            return launch(lightning_tokens_kernel<T>, dim3(s.heads * ((s.vdim + kTokenCols - 1) / kTokenCols), n), dim3(256), lightning_smem_floats(s.state, keep_state) * sizeof(float), ssm_y_,
+                          static_cast<const T *>(proj_), static_cast<long long>(d.proj_cols), static_cast<const float *>(d.decay), s, keep_state, entries_ + entry0);
+        }));
+        return launch(normed_sigmoid_gate_kernel<T>, dim3(rows), dim3(std::min(1024, pad_to((s.inner + 3) / 4, 32))), size_t(s.inner) * sizeof(float), act_, d.mix_out,
+                      static_cast<const float *>(ssm_y_), s.inner, static_cast<const T *>(proj_ + d.off_gate), static_cast<long long>(d.proj_cols), static_cast<const float *>(d.mix_norm),
+                      static_cast<float>(c_.eps));
+    }
+
+    // Calls run(kind, first part, parts) for every stretch of neighbouring parts of one kind.
+    template <typename Kind, typename Run>
+    int runs(const std::vector<Part> &parts, Kind &&kind, Run &&run)
+    {
+        for (size_t i = 0, j; i < parts.size(); i = j) {
+            const auto k = kind(parts[i]);
+            for (j = i + 1; j < parts.size() && kind(parts[j]) == k;) ++j;
+            RC_TRY(run(k, static_cast<int>(i), static_cast<int>(j - i)));
+        }
+        return GPTB200_OK;
+    }
+
+    // ---- wkv: h_ holds the five blends of the normed rows
+    int wkv(const Layer &d, const std::vector<Part> &parts, int rows)
+    {
+        WkvShape s = d.wkv;
+        const int n = s.heads * s.dim;
+        if constexpr (kF32) {
+            s.group = static_cast<long long>(rows) * d.group_cols;
+            s.ld = d.group_cols;
+            for (int g = 0; g < 5; ++g)
+                RC_TRY(run_linear_f32(ctx_, g < 4 ? proj_ + g * s.group : tail_, h_ + g * state_stride_, d.w_in + size_t(g) * d.group_cols * pitch_, rows, g < 4 ? d.group_cols : s.rank_pad, pitch_));
+        } else {
+            s.group = d.group_cols;
+            s.ld = d.proj_cols;
+            Bf16Linear c{};
+            c.M = rows; c.N = d.proj_n; c.K = pitch_; c.a = h_; c.lda = pitch_; c.w = d.w_in; c.out_kind = OUT_BF16; c.out = proj_; c.ldo = d.proj_cols;
+            c.tail = tail_; c.tail_col = d.proj_cols; c.tail_pitch = s.rank_pad;
+            c.group_cols = d.group_cols; c.group_rows = rows_;
+            RC_TRY(run_linear_bf16(ctx_, c));
+        }
+        const auto is_long = [&](const Part &p) { return !kF32 && s.dim <= kWkvMaxDim && p.count >= chunk_rows_; };
+        if constexpr (!kF32) {
+            if (std::any_of(parts.begin(), parts.end(), is_long)) {
+                RC_TRY(launch(wkv_low_rank_kernel, dim3(rows), dim3(std::min(128, pad_to(s.rank_pad, 32))), 0, low_, s.rank_pad, tail_, s.ld_low, s.rank));
+                Bf16Linear c{};
+                c.M = rows; c.N = pad_to(n, 8); c.K = 2 * s.rank_pad; c.a = low_; c.lda = 2 * s.rank_pad; c.w = d.w2; c.out_kind = OUT_F32; c.out = raw_; c.ldo = pad_to(n, 8);
+                RC_TRY(run_linear_bf16(ctx_, c));
+            }
+        }
+        return runs(parts, is_long, [&](bool chunks, int entry0, int count) {
+            if (chunks) return s.dim <= 32 ? wkv_chunks<2>(d, s, parts, entry0, count) : s.dim <= 64 ? wkv_chunks<4>(d, s, parts, entry0, count) : wkv_chunks<8>(d, s, parts, entry0, count);
+            const int threads = std::max(256, pad_to(s.dim, 32));
+            const bool keep_state = wkv_smem_floats(s.dim, s.rank, threads, true) * sizeof(float) <= 200 * 1024;
+            return launch(wkv_tokens_kernel<T>, dim3(s.heads, count), dim3(threads), wkv_smem_floats(s.dim, s.rank, threads, keep_state) * sizeof(float), act_, d.mix_out,
+                          static_cast<const T *>(proj_), static_cast<const float *>(tail_), static_cast<const T *>(d.w2), static_cast<const float *>(d.w0), static_cast<const float *>(d.bonus),
+                          static_cast<const float *>(d.mix_norm), static_cast<float>(c_.eps), s, keep_state, entries_ + entry0);
+        });
+    }
+
+    template <int KT>
+    int wkv_chunks(const Layer &d, const WkvShape &s, const std::vector<Part> &parts, int entry0, int n)
+    {
+        if constexpr (kF32) {
+            return GPTB200_OK;
+        } else {
+            int longest = 0;
+            for (int i = 0; i < n; ++i) longest = std::max(longest, parts[entry0 + i].count);
+            const int tokens = longest > wkv_segment_tokens_ + wkv_segment_tokens_ / 2 ? wkv_segment_tokens_ : pad_to(longest, kWkvChunk), segments = (longest + tokens - 1) / tokens;
+            const size_t smem = wkv_chunk_layout(KT).total, square = size_t(s.dim) * s.dim;
+            float *seg_state = nullptr, *seg_decay = nullptr;
+            const auto chunks = [&](auto kernel, int launched) {
+                return launch(kernel, dim3(s.heads, n, launched), dim3(32 * KT), smem, act_, d.mix_out, proj_, raw_, pad_to(s.heads * s.dim, 8), d.w0, d.bonus, d.mix_norm,
+                              static_cast<float>(c_.eps), s, entries_ + entry0, tokens, segments, seg_state, seg_decay);
+            };
+            if (segments > 1) {
+                const size_t pieces = size_t(n) * s.heads * segments;
+                RC_TRY(scratch(pieces * (square + s.dim)));
+                seg_state = scratch_;
+                seg_decay = scratch_ + pieces * square;
+                RC_TRY(chunks(wkv_chunk_kernel<KT, true>, segments - 1));
+                RC_TRY(launch(wkv_segments_kernel, dim3(s.heads * static_cast<int>((square + 255) / 256), n), dim3(256), 0, seg_state, seg_decay, s, entries_ + entry0, tokens, segments));
+            }
+            return chunks(wkv_chunk_kernel<KT, false>, segments);
+        }
+    }
+
+    int mixer(int layer, const std::vector<Part> &parts, int rows)
+    {
+        const Layer &d = layers_[layer];
+        switch (c_.layers[layer].kind) {
+            case MixerKind::Mamba2: return mamba(d, parts, rows);
+            case MixerKind::Latent: return latent(d, parts, rows);
+            case MixerKind::Grouped: return grouped(d, parts, rows);
+            case MixerKind::Lightning: return lightning(d, parts, rows);
+            default: return wkv(d, parts, rows);
+        }
+    }
+
+    // y_ = gated feed-forward of h_
+    int feed_forward(const Layer &d, int rows)
+    {
+        if constexpr (kF32) {
+            RC_TRY(run_linear_f32(ctx_, glu_, h_, d.w_glu, rows, 2 * d.ff, pitch_));
+            RC_TRY(launch(glu_rows_kernel, dim3(rows), dim3(128), 0, act_, static_cast<const float *>(glu_), d.ff, static_cast<long long>(2 * d.ff), c_.traits.silu_gate));
+        } else {
+            Bf16Linear c{};
+            c.M = rows; c.N = 2 * d.ff; c.K = pitch_; c.a = h_; c.lda = pitch_; c.w = d.w_glu; c.out_kind = c_.traits.silu_gate ? OUT_GLU_SILU : OUT_GLU; c.out = act_; c.ldo = d.ff;
+            RC_TRY(run_linear_bf16(ctx_, c));
+        }
+        return linear_f32(y_, act_, d.w_down, rows, pitch_, d.ff);
+    }
+
+    // h = norm(x + residual_mult * y), or the layer's blends of it; the sum goes to the other buffer of x_ (`at`: the current one)
+    int residual_norm(int rows, int *at, const float *y, const Norm &n, T *h, const Layer *mixes, const int *row_list)
+    {
+        ResidualNorm<T> b{};
+        b.rows = rows; b.width = c_.width; b.pitch = pitch_; b.eps = static_cast<float>(c_.eps); b.mult = static_cast<float>(c_.residual_mult);
+        b.x_in = x_[*at];
+        b.y = y;
+        if (y && !row_list) {
+            *at ^= 1;
+            b.x_out = x_[*at];
+        }
+        b.norm_w = n.w;
+        if (mixes && mixes->mix) {
+            b.mixes = kWkvMixes;
+            b.mix = mixes->mix;
+            b.shift_state = mixes->shift_state;
+            b.mix_stride = state_stride_;
+        }
+        b.h = h;
+        b.entries = entries_; b.row_entry = row_entry_; b.row_list = row_list;
+        b.tile = rows <= 512 || !b.mixes ? 1 : rows <= 2048 ? 4 : 8;
+        return launch(residual_norm_kernel<T>, dim3((rows + b.tile - 1) / b.tile), dim3(row_threads(rows)), 2 * size_t(pitch_) * sizeof(float), b);
+    }
+
+    int rotary_tables(int rows)
+    {
         for (const Rotary &r : rotaries_)
             RC_TRY(launch(rotary_table_kernel, dim3((rows * (r.config.dims / 2) + 127) / 128), dim3(128), 0, table_ + r.table, static_cast<const double *>(r.freq), r.config.dims / 2, r.gain,
                           entries_, row_entry_, rows));
+        return GPTB200_OK;
+    }
+
+    // Norms before the sublayers only: every residual sum happens in the norm that reads it.
+    int kernels_norms_before(const std::vector<Part> &parts, int rows, int n_want)
+    {
+        int at = 0;
+        RC_TRY(launch(embed_pair_rows_kernel<T>, dim3(rows), dim3(row_threads(rows)), 0, x_[0], static_cast<const T *>(embed_), static_cast<float>(c_.embed_scale),
+                      static_cast<const T *>(pairs_), c_.pair_buckets, c_.pair_mul_previous, c_.pair_mul_current, static_cast<const int *>(tokens_), pitch_, previous_state_, entries_, row_entry_));
+        RC_TRY(rotary_tables(rows));
+        const float *y = nullptr;
+        for (size_t i = 0; i < layers_.size(); ++i) {
+            const Layer &d = layers_[i];
+            RC_TRY(residual_norm(rows, &at, y, d.norm1, h_, &d, nullptr));
+            RC_TRY(mixer(static_cast<int>(i), parts, rows));
+            RC_TRY(linear_f32(y_, act_, d.w_o, rows, pitch_, d.mix_out));
+            y = y_;
+            if (d.ff) {
+                RC_TRY(residual_norm(rows, &at, y, d.norm2, h_, nullptr, nullptr));
+                RC_TRY(feed_forward(d, rows));
+            }
+        }
+        if (n_want > 0) {
+            RC_TRY(residual_norm(n_want, &at, y, final_norm_, hw_, nullptr, want_));
+            RC_TRY(linear_f32(logits_, hw_, head_, n_want, vocab_pitch_, pitch_));
+        }
+        return GPTB200_OK;
+    }
+
+    // All kernels of one step; everything that changes from step to step is read from device memory.
+    int kernels(const std::vector<Part> &parts, int rows, int n_want)
+    {
+        if (!norms_around()) return kernels_norms_before(parts, rows, n_want);
+        const float eps = static_cast<float>(c_.eps);
+        RC_TRY(launch(embed_rows_kernel<T>, dim3(rows), dim3(row_threads(rows)), 0, states_, static_cast<const T *>(embed_), static_cast<const int *>(tokens_), pitch_));
+        RC_TRY(rotary_tables(rows));
         for (size_t i = 0; i < layers_.size(); ++i) {
             const Layer &d = layers_[i];
             float *x = x_[i & 1];
             RC_TRY(layer_begin(rows, static_cast<int>(i), h_, nullptr));
-            RC_TRY(c_.layers[i].kind == MixerKind::Mamba2 ? mamba(d, parts, rows) : latent(d, parts, rows));
+            RC_TRY(mixer(static_cast<int>(i), parts, rows));
             RC_TRY(linear_f32(y_, act_, d.w_o, rows, pitch_, d.mix_out));
             const size_t smem = size_t(pitch_) * sizeof(float);
             RC_TRY(launch(sublayer_end_kernel<T>, dim3(rows), dim3(row_threads(rows)), smem, x, static_cast<const float *>(y_), static_cast<const float *>(d.norm1b.w),
                           static_cast<const float *>(d.norm1b.b), static_cast<const float *>(d.norm2.w), static_cast<const float *>(d.norm2.b), h_, c_.width, pitch_, eps));
             if (d.ff) {
-                if constexpr (kF32) {
-                    RC_TRY(run_linear_f32(ctx_, glu_, h_, d.w_glu, rows, 2 * d.ff, pitch_));
-                    RC_TRY(launch(glu_rows_kernel, dim3(rows), dim3(128), 0, act_, static_cast<const float *>(glu_), d.ff, static_cast<long long>(2 * d.ff)));
-                } else {
-                    Bf16Linear c{};
-                    c.M = rows; c.N = 2 * d.ff; c.K = pitch_; c.a = h_; c.lda = pitch_; c.w = d.w_glu; c.out_kind = OUT_GLU; c.out = act_; c.ldo = d.ff;
-                    RC_TRY(run_linear_bf16(ctx_, c));
-                }
-                RC_TRY(linear_f32(y_, act_, d.w_down, rows, pitch_, d.ff));
+                RC_TRY(feed_forward(d, rows));
                 RC_TRY(launch(sublayer_end_kernel<T>, dim3(rows), dim3(row_threads(rows)), smem, x, static_cast<const float *>(y_), static_cast<const float *>(d.norm2b.w),
                               static_cast<const float *>(d.norm2b.b), static_cast<const float *>(nullptr), static_cast<const float *>(nullptr), h_, c_.width, pitch_, eps));
             }
@@ -970,14 +1427,15 @@ private:
 
     std::vector<Layer> layers_;
     std::vector<Rotary> rotaries_;
-    T *embed_ = nullptr, *head_ = nullptr;
+    T *embed_ = nullptr, *head_ = nullptr, *pairs_ = nullptr;
     Norm final_norm_;
     int pitch_ = 0, vocab_pitch_ = 0, side_pitch_ = 0;
     int max_proj_ = 8, max_tail_ = 8, max_act_ = 8, max_ff_ = 8, max_channels_ = 8, max_heads_ = 1, max_inner_ = 8;
-    size_t fixed_state_ = 0, position_bytes_ = 0;
+    int mixes_ = 0, max_raw_ = 0, max_low_ = 0, first_values_cols_ = 0;
+    size_t fixed_state_ = 0, position_bytes_ = 0, previous_state_ = 0;
     std::vector<void *> weights_, work_;
     std::vector<Slot> slots_;
-    int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8, segment_tokens_ = 1024;
+    int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8, segment_tokens_ = 1024, wkv_segment_tokens_ = 256;
     T *expanded_ = nullptr;
     size_t expanded_count_ = 0;
     float *scratch_ = nullptr;
@@ -985,8 +1443,9 @@ private:
     bool generating_ = false;   // launches must serve every length up to the slots' capacities
     int rows_ = 0, wanted_ = 0;
     long long state_stride_ = 0;
-    float *states_ = nullptr, *x_[2] = {nullptr, nullptr}, *y_ = nullptr, *tail_ = nullptr, *dt_ = nullptr, *decay_ = nullptr, *ssm_y_ = nullptr, *glu_ = nullptr, *logits_ = nullptr;
-    T *h_ = nullptr, *proj_ = nullptr, *xbc_ = nullptr, *act_ = nullptr, *hw_ = nullptr;
+    float *states_ = nullptr, *x_[2] = {nullptr, nullptr}, *y_ = nullptr, *tail_ = nullptr, *dt_ = nullptr, *decay_ = nullptr, *ssm_y_ = nullptr, *glu_ = nullptr, *logits_ = nullptr,
+          *raw_ = nullptr;
+    T *h_ = nullptr, *proj_ = nullptr, *xbc_ = nullptr, *act_ = nullptr, *hw_ = nullptr, *first_values_ = nullptr, *low_ = nullptr;
     float2 *table_ = nullptr;
     StepEntry *entries_ = nullptr;
     int *row_entry_ = nullptr, *tokens_ = nullptr, *want_ = nullptr, *history_ = nullptr;

@@ -75,6 +75,39 @@ __global__ void embed_rows_kernel(float *__restrict__ x, const T *__restrict__ t
     for (int d = 4 * threadIdx.x; d < pitch; d += 4 * blockDim.x) store4(dst + d, load4(src + d));
 }
 
+// The same for sequences whose embedding looks one token back: scale * table row + the row of `pairs` that the previous and the
+// current token hash to (a sequence's first token: the row after the hashed ones).  The last token of a portion stays in the
+// sequence's state (`previous`: offset of int [2]).
+template <typename T>
+__global__ void embed_pair_rows_kernel(float *__restrict__ x, const T *__restrict__ table, float scale, const T *__restrict__ pairs, long long buckets, long long mul_previous,
+                                       long long mul_current, const int *__restrict__ tokens, int pitch, size_t previous, const StepEntry *__restrict__ entries,
+                                       const int *__restrict__ row_entry)
+{
+    grid_dependency_wait();
+    grid_dependency_launch();
+    const int row = blockIdx.x, token = tokens[row];
+    const StepEntry e = entries[row_entry[row]];
+    int *state = reinterpret_cast<int *>(e.slot + previous);
+    const T *pair = nullptr;
+    if (buckets > 0) {
+        long long at = buckets;
+        if (row > e.row0 || e.pos0 > 0) at = ((row > e.row0 ? tokens[row - 1] : state[e.parity]) * mul_previous + token * mul_current) % buckets;
+        pair = pairs + at * pitch;
+        if (threadIdx.x == 0 && row == e.row0 + e.count - 1) state[e.parity ^ 1] = token;
+    }
+    const T *src = table + static_cast<long long>(token) * pitch;
+    float *dst = x + static_cast<long long>(row) * pitch;
+    for (int d = 4 * threadIdx.x; d < pitch; d += 4 * blockDim.x) {
+        float4 v = load4(src + d);
+        v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+        if (pair) {
+            const float4 b = load4(pair + d);
+            v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+        }
+        store4(dst + d, v);
+    }
+}
+
 template <typename T>
 struct LayerBegin {
     int rows, width, pitch;
@@ -242,16 +275,139 @@ __global__ void sublayer_end_kernel(float *__restrict__ x, const float *__restri
     }
 }
 
+template <typename T>
+struct ResidualNorm {
+    int rows, width, pitch;
+    float eps, mult;
+    const float *x_in;        // residual stream
+    const float *y;           // result of the sublayer before, null: none
+    float *x_out;             // x_in + mult * y (another buffer than x_in), null: not stored
+    const float *norm_w;      // the factor itself
+    int mixes;                // 0: h is the normed row; else h holds that many blends of it with the previous token's, mix_stride apart
+    const float *mix;         // [mixes][pitch] share of the previous token's
+    size_t shift_state;       // offset in the slot: [2][pitch] floats, the previous token's normed row
+    long long mix_stride;
+    T *h;
+    const StepEntry *entries;
+    const int *row_entry;
+    const int *row_list;      // null: all rows; else only these (no mixes then), h is packed
+    int tile;                 // consecutive rows per block
+};
+
+// Between sublayers without norms of their own results: x += mult * y, h = x / root mean square * weight, and the blends of h with the
+// previous token's where the next mixer reads such.  As in layer_begin_kernel the row before a block's first is computed twice.
+template <typename T>
+__global__ void residual_norm_kernel(const ResidualNorm<T> p)
+{
+    extern __shared__ float sm[];
+    float *x = sm, *before = sm + p.pitch;   // this row / previous row's normed values; every thread touches its own columns only
+    __shared__ float red[32];
+    grid_dependency_wait();
+    grid_dependency_launch();
+
+    auto row_normed = [&](int row, bool write, float *dst) {
+        const long long at = static_cast<long long>(row) * p.pitch;
+        float ss = 0.0f;
+        for (int d = 4 * threadIdx.x; d < p.pitch; d += 4 * blockDim.x) {
+            float4 v = load4(p.x_in + at + d);
+            if (p.y) {
+                const float4 y = load4(p.y + at + d);
+                v.x = fmaf(p.mult, y.x, v.x); v.y = fmaf(p.mult, y.y, v.y); v.z = fmaf(p.mult, y.z, v.z); v.w = fmaf(p.mult, y.w, v.w);
+            }
+            if (write && p.x_out) store4(p.x_out + at + d, v);
+            store4(dst + d, v);
+            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+        const float inv = rsqrtf(block_sum(ss, red) / p.width + p.eps);
+        for (int d = 4 * threadIdx.x; d < p.pitch; d += 4 * blockDim.x) {
+            const float4 v = load4(dst + d), w = load4(p.norm_w + d);
+            store4(dst + d, make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w));
+        }
+    };
+
+    const int first = blockIdx.x * p.tile;
+    if (p.mixes) {
+        const StepEntry e = p.entries[p.row_entry[first]];
+        if (first > e.row0) row_normed(first - 1, false, before);
+    }
+    for (int i = first; i < min(first + p.tile, p.rows); ++i) {
+        const int row = p.row_list ? p.row_list[i] : i;
+        row_normed(row, true, x);
+        T *h = p.h + static_cast<long long>(i) * p.pitch;
+        if (!p.mixes) {
+            for (int d = 4 * threadIdx.x; d < p.pitch; d += 4 * blockDim.x) store4(h + d, load4(x + d));
+            continue;
+        }
+        const StepEntry e = p.entries[p.row_entry[row]];
+        float *state = reinterpret_cast<float *>(e.slot + p.shift_state);
+        const float *old = state + e.parity * p.pitch;
+        float *next = state + (e.parity ^ 1) * p.pitch;
+        const bool from_state = row == e.row0, last = row == e.row0 + e.count - 1;
+        for (int d = 4 * threadIdx.x; d < p.pitch; d += 4 * blockDim.x) {
+            const float4 v = load4(x + d), b = from_state ? load4(old + d) : load4(before + d);
+            for (int k = 0; k < p.mixes; ++k) {
+                const float4 m = load4(p.mix + k * p.pitch + d);
+                store4(h + k * p.mix_stride + d, make_float4(v.x + (b.x - v.x) * m.x, v.y + (b.y - v.y) * m.y, v.z + (b.z - v.z) * m.z, v.w + (b.w - v.w) * m.w));
+            }
+            if (last) store4(next + d, v);
+        }
+        float *t = x;
+        x = before;
+        before = t;
+    }
+}
+
+// A row of a mixer's output divided by its root mean square, times weight, times sigmoid(gate), as T.
+template <typename T>
+__global__ void normed_sigmoid_gate_kernel(T *__restrict__ out, int ld_out, const float *__restrict__ y, int width, const T *__restrict__ gate, long long ld_gate,
+                                           const float *__restrict__ weight, float eps)
+{
+    extern __shared__ float sm[];   // [width], every thread its own columns
+    __shared__ float red[32];
+    grid_dependency_wait();
+    grid_dependency_launch();
+    const long long row = blockIdx.x;
+    y += row * width;
+    gate += row * ld_gate;
+    out += row * ld_out;
+    float ss = 0.0f;
+    if (width % 4 == 0) {
+        for (int i = 4 * threadIdx.x; i < width; i += 4 * blockDim.x) {
+            const float4 v = load4(y + i);
+            store4(sm + i, v);
+            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+        const float inv = rsqrtf(block_sum(ss, red) / width + eps);
+        for (int i = 4 * threadIdx.x; i < width; i += 4 * blockDim.x) {
+            const float4 v = load4(sm + i), w = load4(weight + i), g = load4(gate + i);
+            store4(out + i, make_float4(v.x * inv * w.x * sigmoid_f(g.x), v.y * inv * w.y * sigmoid_f(g.y), v.z * inv * w.z * sigmoid_f(g.z), v.w * inv * w.w * sigmoid_f(g.w)));
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        sm[i] = y[i];
+        ss = fmaf(sm[i], sm[i], ss);
+    }
+    const float inv = rsqrtf(block_sum(ss, red) / width + eps);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) out[i] = from_f<T>(sm[i] * inv * weight[i] * sigmoid_f(to_f(gate[i])));
+}
+
 // Unfused tails of the fp32 products (the bf16 products do these in their epilogues).
-// act[row][j] = gelu(gate) * up from columns in groups of 32 gate | 32 up
-__global__ void glu_rows_kernel(float *__restrict__ act, const float *__restrict__ in, int columns, long long ld_in)
+// act[row][j] = gelu(gate) * up, or silu(gate) * up, from columns in groups of 32 gate | 32 up
+__global__ void glu_rows_kernel(float *__restrict__ act, const float *__restrict__ in, int columns, long long ld_in, bool silu)
 {
     const float *src = in + blockIdx.x * ld_in;
     float *dst = act + static_cast<long long>(blockIdx.x) * columns;
     for (int j = threadIdx.x; j < columns; j += blockDim.x) {
         const int g = (j >> 5) * 64 + (j & 31);
-        dst[j] = gelu_f(src[g]) * src[g + 32];
+        dst[j] = (silu ? silu_f(src[g]) : gelu_f(src[g])) * src[g + 32];
     }
+}
+
+__global__ void silu_columns_kernel(float *__restrict__ x, int columns, long long ld)
+{
+    float *r = x + blockIdx.x * ld;
+    for (int j = threadIdx.x; j < columns; j += blockDim.x) r[j] = silu_f(r[j]);
 }
 
 __global__ void gelu_factor_rows_kernel(float *__restrict__ x, const float *__restrict__ factor, const int *__restrict__ factor_rows, int columns)

@@ -60,7 +60,10 @@ enum OutKind : int {
     OUT_BF16 = 1,       // rounded to bf16; columns from tail_col on stay fp32 and go to `tail`
     OUT_GLU = 2,        // columns come in groups of 32 gate | 32 up: gelu_tanh(gate) * up in bf16, half as many columns
     OUT_GELU_MUL = 3,   // gelu_tanh(out) * factor[factor_rows[row]][column] in bf16
+    OUT_GLU_SILU = 4,   // OUT_GLU with silu(gate) * up
 };
+
+__host__ __device__ constexpr bool is_glu(int out_kind) { return out_kind == OUT_GLU || out_kind == OUT_GLU_SILU; }
 
 struct GemmParams {
     int M, N, K;         // D[M x N] = A[M x K] . B[K x N]
@@ -123,6 +126,10 @@ struct GemmParams {
     const void *factor;         // OUT_GELU_MUL: bf16 table, row pitch factor_pitch (a multiple of 8), 16-byte aligned
     const int *factor_rows;     // row of the table per output row
     int factor_pitch;
+    int silu_cols;              // OUT_BF16: silu is applied to the columns before this one (a multiple of 32)
+    // bf16 form: columns [g * a_group_cols, (g + 1) * a_group_cols) of the output multiply rows from g * a_group_rows on of A -- several
+    // products of differently mixed rows with one weight matrix in one launch.  a_group_cols is a multiple of 256; 0: one group.
+    int a_group_cols, a_group_rows;
 };
 
 constexpr int kTraceSlots = 128;
@@ -198,6 +205,8 @@ __device__ __forceinline__ float gelu_tanh(float x)
     return __fdividef(x, 1.0f + __expf(-2.0f * u));
 }
 
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
+
 // d/dx of gelu_tanh(x) = 0.5 x (1 + tanh u), u = 0.79788456 (x + 0.044715 x^3):
 //   0.5 (1 + t) + 0.5 x (1 - t^2) * 0.79788456 (1 + 3 * 0.044715 x^2),  t = tanh u = 1 - 2 / (1 + exp(2u))
 // (the reference's constants, linear.cu:162-187; exp and division in their fast forms, 1-2 ulp, far inside the 1e-5 bound;
@@ -214,10 +223,14 @@ __device__ __forceinline__ float bf16_hi(uint32_t w) { return __uint_as_float(w 
 
 // One [32 rows x 32 columns] piece of a 16-bit output (this thread: row row0 + lane).  Returns false when there is nothing to stage;
 // otherwise `w` holds the row's 32 bf16 values and `word0` the first 4-byte word of the piece in the output row.  `held`
-// carries the gate columns of OUT_GLU from one piece to the next.
+// carries the gate columns of the gated kinds from one piece to the next.
 __device__ __forceinline__ bool piece_to_bf16(const GemmParams &p, float (&v)[32], float (&held)[32], int row0, int col0, int lane, uint32_t (&w)[16], int &word0)
 {
     word0 = col0 / 2;
+    if (p.bias) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[j] += col0 + j < p.N ? __ldg(p.bias + col0 + j) : 0.0f;
+    }
     if (p.out_kind == OUT_BF16) {
         if (col0 >= p.tail_col) {
             if (row0 + lane < p.M) {
@@ -228,7 +241,11 @@ __device__ __forceinline__ bool piece_to_bf16(const GemmParams &p, float (&v)[32
             }
             return false;
         }
-    } else if (p.out_kind == OUT_GLU) {
+        if (col0 < p.silu_cols) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = silu_fast(v[j]);
+        }
+    } else if (is_glu(p.out_kind)) {
         if (!(col0 & 32)) {
 #pragma unroll
             for (int j = 0; j < 32; ++j) held[j] = v[j];
@@ -236,7 +253,7 @@ __device__ __forceinline__ bool piece_to_bf16(const GemmParams &p, float (&v)[32
         }
         word0 = (col0 - 32) / 4;
 #pragma unroll
-        for (int j = 0; j < 32; ++j) v[j] *= gelu_tanh(held[j]);
+        for (int j = 0; j < 32; ++j) v[j] *= p.out_kind == OUT_GLU ? gelu_tanh(held[j]) : silu_fast(held[j]);
     } else {
         const bool row_ok = row0 + lane < p.M;
         const uint4 *f = reinterpret_cast<const uint4 *>(static_cast<const uint16_t *>(p.factor) +
@@ -375,7 +392,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
             for (long long w = blockIdx.x; ok && w < num_items; w += gridDim.x) {
                 int tm, tn, kb0, kb1, split;
                 decode(w, tm, tn, kb0, kb1, split);
-                const int m0 = tm * kBM, n0 = tn * BN;
+                const int n0 = tn * BN, m0 = tm * kBM + (p.a_group_cols ? n0 / p.a_group_cols * p.a_group_rows : 0);
                 for (int kb = kb0; kb < kb1; ++kb, ++it) {
                     const int s = it % STAGES;
                     const uint32_t ph = (it / STAGES) & 1u;
@@ -497,7 +514,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
         uint32_t g = 0;
         bool ok = true;
 
-        float held[32];   // gate columns of OUT_GLU
+        float held[32];   // gate columns of the gated kinds
         // bias / GELU, staging, TMA store of one [32 rows x 32 cols] piece of the tile
         auto emit = [&](float (&v)[32], int row0, int col0, int split) {
             if constexpr (!A_MN && !B_MN && !X3) {

@@ -543,7 +543,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                 const int z = p.batches > 0 ? tn / p.tiles_n : 0;                     // batched form: the tile columns of all batches are numbered through
                 if (p.batches > 0) tn -= z * p.tiles_n;
                 const int zi = p.batches > 0 ? z % p.batch_inner : 0, zo = p.batches > 0 ? z / p.batch_inner : 0;
-                const int m0 = tm2 * 2 * kBM + static_cast<int>(rank) * kBM;          // the rows this CTA owns
+                const int m0 = tm2 * 2 * kBM + static_cast<int>(rank) * kBM           // the rows this CTA owns
+                               + (p.a_group_cols ? tn * BN / p.a_group_cols * p.a_group_rows : 0);
                 const int n0 = tn * BN + static_cast<int>(rank) * (p.mma_n ? p.mma_n / 2 : C::kBRows);   // the half of B this CTA loads
                 for (int kb = kb0; kb < kb1; ++kb, ++it) {
                     const int s = it % STAGES;
@@ -730,7 +731,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
         const uint32_t leader_tmem_empty[2] = {ptx::map_to_cta(tmem_empty_bar(0), 0u), ptx::map_to_cta(tmem_empty_bar(1), 0u)};
 
         int ezi = 0, ezo = 0;   // batched form: batch coordinates of the tile being written
-        float held[32];   // bf16 form: gate columns of OUT_GLU
+        float held[32];   // bf16 form: gate columns of the gated kinds
         // bias_lane: bias[col0 + lane], fetched when the tile was started
         auto emit = [&](float (&v)[32], int row0, int col0, float bias_lane) {
             if constexpr (!A_MN && !B_MN && !X3) {

@@ -28,6 +28,10 @@ struct GemvParams {
     const uint16_t *factor;
     const int *factor_rows;
     int factor_pitch;
+    const float *bias;      // null: none
+    int silu_cols;          // OUT_BF16: silu is applied to the columns before this one
+    int group_cols;         // columns per group (a multiple of 64; >= N: one group); blockIdx.y counts the groups,
+    long long group_x;      //   whose rows of x lie this many elements apart
     int k_warps;            // one row: warps of a block that share a pair of weight rows (1, 2, 4, 8)
 };
 
@@ -41,18 +45,22 @@ __device__ __forceinline__ float bf16_round_store(uint16_t *dst, float v)
     return v;
 }
 
-// One finished value (OUT_GLU: `v` is the gate and `u` the up column of the pair).
+// One finished value (gated kinds: `v` is the gate and `u` the up column of the pair).
 __device__ __forceinline__ void gemv_emit(const GemvParams &p, int m, int n, float v, float u)
 {
+    if (p.bias) {
+        v += __ldg(p.bias + n);
+        if (is_glu(p.out_kind)) u += __ldg(p.bias + n + 32);
+    }
     if (p.out_kind == OUT_F32) {
         static_cast<float *>(p.out)[m * p.ldo + n] = v;
     } else if (p.out_kind == OUT_BF16) {
         if (n >= p.tail_col)
             p.tail[static_cast<long long>(m) * p.tail_pitch + (n - p.tail_col)] = v;
         else
-            bf16_round_store(static_cast<uint16_t *>(p.out) + m * p.ldo + n, v);
-    } else if (p.out_kind == OUT_GLU) {
-        bf16_round_store(static_cast<uint16_t *>(p.out) + m * p.ldo + (n >> 6) * 32 + (n & 31), gelu_tanh(v) * u);
+            bf16_round_store(static_cast<uint16_t *>(p.out) + m * p.ldo + n, n < p.silu_cols ? silu_fast(v) : v);
+    } else if (is_glu(p.out_kind)) {
+        bf16_round_store(static_cast<uint16_t *>(p.out) + m * p.ldo + (n >> 6) * 32 + (n & 31), (p.out_kind == OUT_GLU ? gelu_tanh(v) : silu_fast(v)) * u);
     } else {
         const float f = __uint_as_float(static_cast<uint32_t>(p.factor[static_cast<long long>(p.factor_rows[m]) * p.factor_pitch + n]) << 16);
         bf16_round_store(static_cast<uint16_t *>(p.out) + m * p.ldo + n, gelu_tanh(v) * f);
@@ -73,7 +81,7 @@ __device__ __forceinline__ float dot8(const uint4 &a, const uint4 &b, float acc)
 // The two weight rows of pair `i`: adjacent rows, or a gate row and its up row (groups of 32 gate | 32 up).
 __device__ __forceinline__ void gemv_pair(int i, int out_kind, int &ra, int &rb)
 {
-    if (out_kind == OUT_GLU) {
+    if (is_glu(out_kind)) {
         ra = (i >> 5) * 64 + (i & 31);
         rb = ra + 32;
     } else {
@@ -91,7 +99,9 @@ gemv_bf16_kernel(const GemvParams p)
     __shared__ float2 parts[SHARED ? kGemvThreads / 32 : 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int chunks = p.K >> 3;
-    const int pairs = p.out_kind == OUT_GLU ? p.N / 2 : (p.N + 1) / 2;
+    const int n0 = blockIdx.y * p.group_cols, N = min(p.N - n0, p.group_cols);   // this group's columns
+    const uint16_t *w = p.w + static_cast<long long>(n0) * p.K, *x = p.x + blockIdx.y * p.group_x;
+    const int pairs = is_glu(p.out_kind) ? N / 2 : (N + 1) / 2;
     const int k_warps = SHARED ? p.k_warps : 1;
     const int per_block = (kGemvThreads / 32) / k_warps, stride = gridDim.x * per_block;
     int pair = blockIdx.x * per_block + warp / k_warps;
@@ -102,19 +112,19 @@ gemv_bf16_kernel(const GemvParams p)
     auto fetch = [&](int i, int c0) {
         int ra, rb;
         gemv_pair(i, p.out_kind, ra, rb);
-        const uint4 *a = reinterpret_cast<const uint4 *>(p.w + static_cast<long long>(ra) * p.K);
-        const uint4 *b = reinterpret_cast<const uint4 *>(p.w + static_cast<long long>(rb) * p.K);
+        const uint4 *a = reinterpret_cast<const uint4 *>(w + static_cast<long long>(ra) * p.K);
+        const uint4 *b = reinterpret_cast<const uint4 *>(w + static_cast<long long>(rb) * p.K);
 #pragma unroll
         for (int u = 0; u < kGemvUnroll; ++u) {
             const int c = c0 + u * 32 + lane;
             wa[u] = c < end ? __ldg(a + c) : make_uint4(0u, 0u, 0u, 0u);
-            wb[u] = c < end && rb < p.N ? __ldg(b + c) : make_uint4(0u, 0u, 0u, 0u);
+            wb[u] = c < end && rb < N ? __ldg(b + c) : make_uint4(0u, 0u, 0u, 0u);
         }
     };
     if (pair < pairs) fetch(pair, begin);
     grid_dependency_wait();
     grid_dependency_launch();
-    for (int i = threadIdx.x; i < chunks; i += kGemvThreads) gemv_x[i] = *(reinterpret_cast<const uint4 *>(p.x) + i);
+    for (int i = threadIdx.x; i < chunks; i += kGemvThreads) gemv_x[i] = *(reinterpret_cast<const uint4 *>(x) + i);
     __syncthreads();
     for (; pair < pairs; pair += stride) {
         float sa = 0.0f, sb = 0.0f;
@@ -144,8 +154,8 @@ gemv_bf16_kernel(const GemvParams p)
             continue;
         }
         if (lane == 0) {
-            gemv_emit(p, 0, ra, sa, sb);
-            if (p.out_kind != OUT_GLU && rb < p.N) gemv_emit(p, 0, rb, sb, 0.0f);
+            gemv_emit(p, 0, n0 + ra, sa, sb);
+            if (!is_glu(p.out_kind) && rb < N) gemv_emit(p, 0, n0 + rb, sb, 0.0f);
         }
     }
     if (SHARED) {
@@ -159,14 +169,14 @@ gemv_bf16_kernel(const GemvParams p)
             }
             int ra, rb;
             gemv_pair(done, p.out_kind, ra, rb);
-            gemv_emit(p, 0, ra, sa, sb);
-            if (p.out_kind != OUT_GLU && rb < p.N) gemv_emit(p, 0, rb, sb, 0.0f);
+            gemv_emit(p, 0, n0 + ra, sa, sb);
+            if (!is_glu(p.out_kind) && rb < N) gemv_emit(p, 0, n0 + rb, sb, 0.0f);
         }
     }
 }
 
 // Two to eight rows: the same stream of weights as the A operand of m16n8k16 products (16 weight rows, up to eight rows of x).  A
-// block takes TILES x 16 weight rows (OUT_GLU: 16 gate rows and their 16 up rows) and its eight warps share k, so no value of x is read
+// block takes TILES x 16 weight rows (gated kinds: 16 gate rows and their 16 up rows) and its eight warps share k, so no value of x is read
 // twice by a block and x comes straight from L2.  The order of k inside a block
 // of 32 is permuted alike on both sides so that a lane loads 16 contiguous bytes of a row: piece c of a block (8 values) feeds
 // two products, values 0-3 the first and 4-7 the second.
@@ -186,11 +196,13 @@ gemv_bf16_mma_kernel(const GemvParams p)
     __shared__ float sums[8 * TILES * 16 * 8];   // [warp][weight row][row of x]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, c = lane & 3;
+    const int n0 = blockIdx.y * p.group_cols, N = min(p.N - n0, p.group_cols);   // this group's columns
+    const uint16_t *w = p.w + static_cast<long long>(n0) * p.K;
     // weight rows of the block's tiles
     int row[TILES];
 #pragma unroll
     for (int t = 0; t < TILES; ++t)
-        row[t] = p.out_kind == OUT_GLU ? (blockIdx.x >> 1) * 64 + (blockIdx.x & 1) * 16 + t * 32 : (blockIdx.x * TILES + t) * 16;
+        row[t] = is_glu(p.out_kind) ? (blockIdx.x >> 1) * 64 + (blockIdx.x & 1) * 16 + t * 32 : (blockIdx.x * TILES + t) * 16;
     const int blocks = (p.K + 31) / 32, per_warp = (blocks + 7) / 8;
     const int first = warp * per_warp, end = min(blocks, first + per_warp);
     uint4 wv[kGemvMmaUnroll][TILES][2];
@@ -203,7 +215,7 @@ gemv_bf16_mma_kernel(const GemvParams p)
 #pragma unroll
                 for (int half = 0; half < 2; ++half) {
                     const int r = row[t] + g + 8 * half;
-                    wv[u][t][half] = blk + u < end && k < p.K && r < p.N ? __ldg(reinterpret_cast<const uint4 *>(p.w + static_cast<long long>(r) * p.K + k)) : make_uint4(0u, 0u, 0u, 0u);
+                    wv[u][t][half] = blk + u < end && k < p.K && r < N ? __ldg(reinterpret_cast<const uint4 *>(w + static_cast<long long>(r) * p.K + k)) : make_uint4(0u, 0u, 0u, 0u);
                 }
         }
     };
@@ -212,7 +224,7 @@ gemv_bf16_mma_kernel(const GemvParams p)
     grid_dependency_launch();
     float acc[TILES][4] = {};
     const bool live = g < p.M;   // this lane's row of x
-    const uint16_t *xs = p.x + (live ? g : 0) * p.ldx + c * 8;
+    const uint16_t *xs = p.x + blockIdx.y * p.group_x + (live ? g : 0) * p.ldx + c * 8;
     for (int blk = first; blk < end; blk += kGemvMmaUnroll) {
         if (blk > first) fetch(blk);
         uint4 xv[kGemvMmaUnroll];
@@ -235,7 +247,7 @@ gemv_bf16_mma_kernel(const GemvParams p)
 #pragma unroll
         for (int i = 0; i < 4; ++i) sums[(warp * TILES * 16 + t * 16 + g + (i >> 1) * 8) * 8 + 2 * c + (i & 1)] = acc[t][i];
     __syncthreads();
-    const int outputs = p.out_kind == OUT_GLU ? 128 : TILES * 128;
+    const int outputs = is_glu(p.out_kind) ? 128 : TILES * 128;
     for (int i = threadIdx.x; i < outputs; i += kGemvThreads) {
         const int r = i >> 3, m = i & 7;
         if (m >= p.M) continue;
@@ -243,10 +255,10 @@ gemv_bf16_mma_kernel(const GemvParams p)
 #pragma unroll
         for (int w = 0; w < 8; ++w) {
             v += sums[(w * TILES * 16 + r) * 8 + m];
-            if (TILES == 2 && p.out_kind == OUT_GLU) up += sums[(w * TILES * 16 + 16 + r) * 8 + m];
+            if (TILES == 2 && is_glu(p.out_kind)) up += sums[(w * TILES * 16 + 16 + r) * 8 + m];
         }
-        const int n = p.out_kind == OUT_GLU ? row[0] + r : blockIdx.x * TILES * 16 + r;
-        if (n < p.N) gemv_emit(p, m, n, v, up);
+        const int n = is_glu(p.out_kind) ? row[0] + r : blockIdx.x * TILES * 16 + r;
+        if (n < N) gemv_emit(p, m, n0 + n, v, up);
     }
 }
 

@@ -40,6 +40,12 @@ struct Json {
         if (!(v >= 1.0 && v <= 2147483647.0) || v != static_cast<double>(static_cast<long long>(v))) throw std::runtime_error("'" + key + "' is not a positive integer");
         return static_cast<int>(v);
     }
+    bool flag(const std::string &key) const
+    {
+        const Json &v = at(key);
+        if (v.kind != Bool) throw std::runtime_error("'" + key + "' is not true or false");
+        return v.boolean;
+    }
     const std::string &str(const std::string &key) const
     {
         const Json &v = at(key);

@@ -10,10 +10,17 @@
 namespace gptb200 {
 namespace dec {
 
-struct MambaShape {
-    int heads, vdim, state, groups, taps, norm_groups;
-    int inner, channels;        // heads * vdim; inner + 2 * groups * state
-    size_t conv_state, ssm_state;   // offsets in the slot
+// A state of [state x vdim] per head; rows of values | state inputs | state outputs: [x: inner | B: groups * state | C: groups * state].
+struct RecurrentShape {
+    int heads, vdim, state, groups;
+    int inner;                  // heads * vdim
+    size_t ssm_state;           // offset in the slot: [2][heads][state][vdim] floats
+};
+
+struct MambaShape : RecurrentShape {
+    int taps, norm_groups;
+    int channels;               // inner + 2 * groups * state
+    size_t conv_state;          // offset in the slot
 };
 
 // Convolution + silu of one channel per thread; blocks beyond the channels compute the step sizes and log-decays.
@@ -60,7 +67,7 @@ __global__ void mamba_conv_kernel(T *__restrict__ xbc, int ld_xbc, float *__rest
 // The recurrence token by token: one block per (head, entry), state in shared memory.  y [rows][inner] fp32.
 template <typename T>
 __global__ void mamba_scan_kernel(float *__restrict__ y, const T *__restrict__ xbc, int ld_xbc, const float *__restrict__ dt, const float *__restrict__ log_decay,
-                                  const float *__restrict__ d_skip, const MambaShape s, const StepEntry *__restrict__ entries)
+                                  const float *__restrict__ d_skip, const RecurrentShape s, const StepEntry *__restrict__ entries)
 {
     extern __shared__ float sm[];
     const int P = s.vdim, N = s.state, h = blockIdx.x;

@@ -1,4 +1,5 @@
-// Mamba-2 recurrence over prompts: the state-space duality form in chunks of 64 tokens, on tensor cores.
+// Recurrences with one decay per head and token (Mamba-2; linear attention with constant decays: steps of one, no skip) over prompts: the
+// state-space duality form in chunks of 64 tokens, on tensor cores.
 //
 // With a_t the running sum of log-decays inside a chunk and S the state before it,
 //   y_t = exp(a_t) C_t S + sum_{s <= t} exp(a_t - a_s) dt_s (C_t . B_s) x_s + D x_t
@@ -78,11 +79,12 @@ __host__ __device__ inline int chunk_smem_bytes(int state)
 
 // SEGMENT_STATES: only what a segment adds to the state, from zero, into segment_state [entry][head][segment][state][vdim] and the
 // segment's decay into segment_decay [entry][head][segment]; the last segment is left out.  Otherwise outputs and, in the last
-// segment, the request's new state.  grid: (heads * column slices, entries, segments)
+// segment, the request's new state.  dt null: steps of one; ld_decay: row pitch of log_decay (0: constant decays); d_skip null: none.
+// grid: (heads * column slices, entries, segments)
 template <bool SEGMENT_STATES>
 __global__ void __launch_bounds__(kChunkThreads, 2)
-mamba_chunk_kernel(float *__restrict__ y, const __nv_bfloat16 *__restrict__ xbc, int ld_xbc, const float *__restrict__ dt, const float *__restrict__ log_decay,
-                   const float *__restrict__ d_skip, const MambaShape s, const StepEntry *__restrict__ entries, int segment_tokens, int max_segments, float *__restrict__ segment_state,
+mamba_chunk_kernel(float *__restrict__ y, const __nv_bfloat16 *__restrict__ xbc, int ld_xbc, const float *__restrict__ dt, const float *__restrict__ log_decay, int ld_decay,
+                   const float *__restrict__ d_skip, const RecurrentShape s, const StepEntry *__restrict__ entries, int segment_tokens, int max_segments, float *__restrict__ segment_state,
                    float *__restrict__ segment_decay)
 {
     using namespace mma16;
@@ -158,9 +160,9 @@ mamba_chunk_kernel(float *__restrict__ y, const __nv_bfloat16 *__restrict__ xbc,
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const int t = chunk * kChunk + 2 * lane + i;
-            const long long at = static_cast<long long>(first_row + t) * s.heads + h;
-            ld[i] = t < count ? log_decay[at] * kLog2e : 0.0f;
-            sd[i] = t < count ? dt[at] : 0.0f;
+            const long long row = first_row + t;
+            ld[i] = t < count ? log_decay[row * ld_decay + h] * kLog2e : 0.0f;
+            sd[i] = t >= count ? 0.0f : dt ? dt[row * s.heads + h] : 1.0f;
         }
     };
     auto finish_tokens = [&](int b) {
@@ -207,7 +209,7 @@ mamba_chunk_kernel(float *__restrict__ y, const __nv_bfloat16 *__restrict__ xbc,
         }
     }
     if (warp == 7) finish_tokens(0);
-    const float skip = d_skip[h];
+    const float skip = d_skip ? d_skip[h] : 0.0f;
     const int chunks = (count + kChunk - 1) / kChunk;
     for (int ch = 0; ch < chunks; ++ch) {
         const int b = ch & 1, t0 = ch * kChunk;

@@ -124,7 +124,7 @@ def _decoder(folder: str, config: dict, dtype: str, device: int, stream: int | N
 
 
 # architecture name in config.json -> class
-REGISTRY = {"Budurax": _decoder, "GPT2": Gpt2}
+REGISTRY = {"Budurax": _decoder, "Lutelorn": _decoder, "GPT2": Gpt2}
 
 
 def load_model(folder: str, dtype: str = "bfloat16", device: int = 0, stream: int | None = None):

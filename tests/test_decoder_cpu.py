@@ -75,7 +75,7 @@ def test_rotation_frequencies(decoder, rot):
 
 def test_registry_names_are_architectures_of_the_library(decoder, tmp_path):
     from gpt_b200 import serving
-    assert set(serving.REGISTRY) == {"Budurax", "GPT2"}
+    assert set(serving.REGISTRY) == {"Budurax", "Lutelorn", "GPT2"}
     (tmp_path / "config.json").write_text('{"architecture": "Other"}')
     with pytest.raises(ValueError, match="Other"):
         serving.load_model(str(tmp_path))
