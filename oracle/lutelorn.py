@@ -25,8 +25,11 @@ def bigram_rows(tokens, buckets, mul_prev, mul_cur):
 
 
 def embedding(tokens, w, e):
+    x = w["embed"][tokens] * e["scale"]
+    if "bigram" not in e:
+        return x
     b = e["bigram"]
-    return w["embed"][tokens] * e["scale"] + w["bigram"][bigram_rows(tokens, b["buckets"], b["mul_prev"], b["mul_cur"])]
+    return x + w["bigram"][bigram_rows(tokens, b["buckets"], b["mul_prev"], b["mul_cur"])]
 
 
 def previous(h):
@@ -62,8 +65,10 @@ def rotate_neighbours(x, rot):
 
 
 def capped_attention(q, k, v, scale, cap):
-    """q / k [T, d], v [T, e]: softmax over the keys up to the query's own of cap tanh(score / cap)."""
-    s = cap * np.tanh((q @ k.T) * scale / cap)
+    """q / k [T, d], v [T, e]: softmax over the keys up to the query's own of cap tanh(score / cap); no cap: of the scores."""
+    s = (q @ k.T) * scale
+    if cap is not None:
+        s = cap * np.tanh(s / cap)
     s = np.where(np.tril(np.ones_like(s)) > 0, s, -np.inf)
     p = np.exp(s - s.max(-1, keepdims=True))
     return (p / p.sum(-1, keepdims=True)) @ v
@@ -77,10 +82,12 @@ def attention(h, w, p, m, first_values):
     """-> (output, this layer's own values [T, kv_heads, vdim] before any mixing)."""
     H, G, d, e = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q, k, v = ((h @ w[p + n].T + w[p + n + ".b"]).reshape(-1, heads, size) for n, heads, size in (("q", H, d), ("k", G, d), ("v", G, e)))
-    q, k, own = rotate_neighbours(q, m["rot"]), rotate_neighbours(k, m["rot"]), v
+    own = v
+    if "rot" in m:
+        q, k = rotate_neighbours(q, m["rot"]), rotate_neighbours(k, m["rot"])
     if m.get("v_mix") and first_values is not None:
         v = mixed_values(v, first_values, float(np.asarray(w[p + "vmix"]).reshape(())))
-    out = np.stack([capped_attention(q[:, n], k[:, n // (H // G)], v[:, n // (H // G)], m["scale"], m["softcap"]) for n in range(H)], 1)
+    out = np.stack([capped_attention(q[:, n], k[:, n // (H // G)], v[:, n // (H // G)], m["scale"], m.get("softcap")) for n in range(H)], 1)
     return (out.reshape(len(h), H * e) * sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T, own
 
 

@@ -3,6 +3,7 @@ import numpy as np
 import pytest
 
 import decoder_models as dm
+from decoder_models import load, whole
 from oracle import budurax
 
 pytestmark = pytest.mark.gpu
@@ -45,30 +46,6 @@ def build(layers, overrides, other, seed=1):
             if name.split(".", 1)[-1] == key:
                 w[name] = np.eye(1, len(w[name]))[0].astype(np.float32) if isinstance(value, str) else np.full_like(w[name], value)
     return c, w
-
-
-def load(tmp_path, c, w, dtype):
-    from gpt_b200 import serving
-    return serving.load_model(dm.save(tmp_path / "model", c, w), dtype)
-
-
-def portions(model, seq, tokens, cuts):
-    """Logits of all rows, the tokens fed in portions of the given sizes (the last size repeats)."""
-    out, at, i = [], 0, 0
-    while at < len(tokens):
-        n = min(cuts[min(i, len(cuts) - 1)], len(tokens) - at)
-        out.append(model.step([(seq, tokens[at:at + n])], range(n)))
-        at += n
-        i += 1
-    return np.concatenate(out)
-
-
-def whole(model, tokens, cuts=(1 << 20,), max_len=None):
-    seq = model.open(max_len or len(tokens))
-    try:
-        return portions(model, seq, tokens, cuts)
-    finally:
-        model.close(seq)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
