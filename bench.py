@@ -1018,8 +1018,48 @@ def decoder_folder(torch, dev, folder, z):
         for n in ("norm1", "norm1b", "norm2", "norm2b"):
             shapes += [(p + n, (W,)), (p + n + ".b", (W,))]
     shapes += [("final.norm", (W,)), ("final.norm.b", (W,)), ("head", (z["vocab"], W))]
+    return write_decoder(torch, dev, folder, dict(architecture="Budurax", width=W, vocab=z["vocab"], norm=dict(eps=1e-5), token_side=dict(dim=z["side"]), layers=layers), shapes)
+
+
+# Lutelorn models of the widths, feed-forward widths and numbers of layers of DECODER_SIZES: lightning, wkv, lightning, attention, ...
+LUTELORN_SIZES = {
+    "w768": dict(width=768, ff=3072, heads=12, kv_heads=4, dim=64, rot_dim=32, light_heads=12, light_dim=64, wkv_heads=12, wkv_dim=64, rank=32, layers=12, vocab=50304),
+    "w2048": dict(width=2048, ff=8192, heads=16, kv_heads=4, dim=128, rot_dim=64, light_heads=16, light_dim=128, wkv_heads=32, wkv_dim=64, rank=64, layers=8, vocab=50304),
+    "w4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, rot_dim=64, light_heads=32, light_dim=128, wkv_heads=64, wkv_dim=64, rank=128, layers=4, vocab=50304),
+}
+
+
+def lutelorn_folder(torch, dev, folder, z):
+    """Writes config.json and model.safetensors of a Lutelorn model of size z with random bf16 weights (generated on the GPU)."""
+    W, layers, buckets = z["width"], [], 65521
+    shapes = [("embed", (z["vocab"], W)), ("bigram", (buckets + 1, W))]
+    for i in range(z["layers"]):
+        p, m = f"l{i}.", f"l{i}.mix."
+        if i % 4 == 3:
+            H, G, d = z["heads"], z["kv_heads"], z["dim"]
+            layers.append(dict(type="attention", mixer=dict(heads=H, kv_heads=G, dim=d, vdim=d, scale=d ** -0.5, softcap=40.0, v_mix=True, rot=dict(base=500000.0, dims=z["rot_dim"]))))
+            shapes += [(m + "q", (H * d, W)), (m + "q.b", (H * d,)), (m + "k", (G * d, W)), (m + "k.b", (G * d,)), (m + "v", (G * d, W)), (m + "v.b", (G * d,)), (m + "vmix", (1,)), (m + "g", (H * d, W)),
+                       (m + "o", (W, H * d))]
+        elif i % 4 == 1:
+            n = z["wkv_heads"] * z["wkv_dim"]
+            layers.append(dict(type="wkv", mixer=dict(heads=z["wkv_heads"], dim=z["wkv_dim"])))
+            shapes += [(m + x, (n, W)) for x in "rkvg"] + [(m + "mu." + x, (W,)) for x in "rkvgw"]
+            shapes += [(m + "w1", (z["rank"], W)), (m + "w2", (n, z["rank"])), (m + "w0", (n,)), (m + "u", (z["wkv_heads"], z["wkv_dim"])), (m + "norm", (n,)), (m + "o", (W, n))]
+        else:
+            H, d = z["light_heads"], z["light_dim"]
+            layers.append(dict(type="lightning", mixer=dict(heads=H, dim=d, vdim=d, decay=[1.0 - 2.0 ** (-1 - 8.0 * h / H) for h in range(H)])))
+            shapes += [(m + x, (H * d, W)) for x in "qkvg"] + [(m + "norm", (H * d,)), (m + "o", (W, H * d))]
+        layers[-1]["mlp"] = dict(kind="dense", ff=z["ff"])
+        shapes += [(p + "norm1", (W,)), (p + "norm2", (W,)), (p + "mlp.gate", (z["ff"], W)), (p + "mlp.up", (z["ff"], W)), (p + "mlp.down", (W, z["ff"]))]
+    shapes += [("final.norm", (W,)), ("head", (z["vocab"], W))]
+    config = dict(architecture="Lutelorn", width=W, vocab=z["vocab"], norm=dict(eps=1e-5), residual_mult=0.5, embedding=dict(scale=1.0, bigram=dict(buckets=buckets, mul_prev=31337, mul_cur=7919)),
+                  layers=layers)
+    return write_decoder(torch, dev, folder, config, shapes, norms_around_zero=True)
+
+
+def write_decoder(torch, dev, folder, config, shapes, norms_around_zero=False):
     with open(os.path.join(folder, "config.json"), "w") as f:
-        json.dump(dict(architecture="Budurax", width=W, vocab=z["vocab"], norm=dict(eps=1e-5), token_side=dict(dim=z["side"]), layers=layers), f)
+        json.dump(config, f)
     header, at = {}, 0
     for name, shape in shapes:
         n = 2
@@ -1035,24 +1075,26 @@ def decoder_folder(torch, dev, folder, z):
             t = torch.randn(shape, device=dev, generator=gen) * (shape[1] ** -0.5 if len(shape) == 2 else 0.1)
             if name.endswith("dwa"):
                 t[-1] += 1.0
-            if name.endswith("norm") or name[-6:-1] == ".norm" or name.endswith(("norm1b", "norm2b")):
+            if name.endswith("mix.norm") or (not norms_around_zero and (name.endswith("norm") or name[-6:-1] == ".norm" or name.endswith(("norm1b", "norm2b")))):
                 t += 1.0
+            if name.endswith(".w0"):
+                t -= 2.0
             f.write(t.bfloat16().view(torch.int16).cpu().numpy().tobytes())
     return at
 
 
-def decoder_record(torch, dev, sizes, prompts=(2048, 8192), context=1024, batches=(1, 8), steps=64, reps=3, gpt2=True):
-    """Prompt and decoding throughput of Budurax models (bf16) of real layer sizes through the public API (gpt_b200.serving.load_model:
-    step / generate, token ids from and to the host), and of GPT-2 (fp32, TF32 products) with the same width, feed-forward
+def decoder_record(torch, dev, sizes, prompts=(2048, 8192), context=1024, batches=(1, 8), steps=64, reps=3, gpt2=True, table=None, folder_of=None):
+    """Prompt and decoding throughput of decoder models (bf16; Budurax unless `table` and `folder_of` name another) of real layer sizes
+    through the public API (gpt_b200.serving.load_model: step / generate, token ids from and to the host), and of GPT-2 (fp32, TF32 products) with the same width, feed-forward
     width and number of layers: a forward pass over 8 x 1024 tokens, and its CUDA-graph-replayed decode step."""
     import gpt_b200
     from gpt_b200 import serving
     out, launches = {}, 0
     for name in sizes:
-        z = DECODER_SIZES[name]
+        z = (table or DECODER_SIZES)[name]
         rec = {"parameters_bytes": 0, "prompt": {}, "decode": {}}
         with tempfile.TemporaryDirectory() as folder:
-            rec["parameters_bytes"] = decoder_folder(torch, dev, folder, z)
+            rec["parameters_bytes"] = (folder_of or decoder_folder)(torch, dev, folder, z)
             stream = torch.cuda.Stream()
             model = serving.load_model(folder, "bfloat16", dev.index, stream.cuda_stream)
         gen = torch.Generator().manual_seed(2)
@@ -1200,20 +1242,27 @@ def decoder_gpt2(torch, dev, z, context, batches, steps, reps):
 
 
 def run_decoder(args):
-    """--workload decoder: see decoder_record; the JSON `value` is the prompt throughput of the middle size at 8192 tokens."""
+    """--workload decoder (Budurax) and lutelorn: see decoder_record; the JSON `value` is the prompt throughput of the middle size at 8192 tokens."""
     import torch
     torch.cuda.set_device(0)
     dev = torch.device("cuda", 0)
     sampler = ClockSampler(0)
     t_begin = time.time()
     sizes = args.decoder_sizes.split(",")
-    rec = decoder_record(torch, dev, sizes, gpt2=not args.profile)
+    if args.workload == "lutelorn":
+        rec = decoder_record(torch, dev, sizes, gpt2=False, table=LUTELORN_SIZES, folder_of=lutelorn_folder)
+        beside = {} if args.profile else decoder_record(torch, dev, sizes, gpt2=False)["sizes"]
+        for name, r in beside.items():
+            rec["sizes"][name]["budurax"] = r
+        what, table = "Lutelorn decoder models with real layer sizes, random weights: prompts and CUDA-graph decoding through gpt_b200.serving; Budurax of equal width beside them", LUTELORN_SIZES
+    else:
+        rec = decoder_record(torch, dev, sizes, gpt2=not args.profile)
+        what, table = "Budurax decoder models with real layer sizes, random weights: prompts and CUDA-graph decoding through gpt_b200.serving; GPT-2 of equal width beside them", DECODER_SIZES
     clocks = sampler.stop(t_begin, time.time())
     main_rec = rec["sizes"]["w2048" if "w2048" in sizes else sizes[0]]["prompt"]["8192"]
     out = dict(metric="decoder_prompt_tokens_per_s", value=main_rec["tokens_per_s"], unit="tokens/s", n_gpus=1, steps=3, warmup=1, ms_per_step=main_rec["ms"], higher_is_better=True,
                scaling="weak", vs_baseline=None, dtype="bf16", data="synthetic", impl="ours",
-               config=dict(workload="Budurax decoder models with real layer sizes, random weights: prompts and CUDA-graph decoding through gpt_b200.serving; GPT-2 of equal width beside them",
-                           sizes={k: DECODER_SIZES[k] for k in sizes}, l2="weights and activations of a step (> 400 MB) exceed the 126 MB L2 at w2048 and w4096"),
+               config=dict(workload=what, sizes={k: table[k] for k in sizes}, l2="weights and activations of a step (> 400 MB) exceed the 126 MB L2 at w2048 and w4096"),
                sizes=rec["sizes"], gpu_launches=rec["gpu_launches"], clocks=clocks)
     print(json.dumps(out), flush=True)
 
@@ -1319,9 +1368,9 @@ def main():
     ap.add_argument("--cpu-rows", type=int, default=256, help="rows of the workload the cpu_baseline leg runs")
     ap.add_argument("--ref-rows", type=int, default=32, help="rows per step of the --impl reference arm")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--workload", choices=["ffn", "train", "decode", "generate", "attention", "decoder"], default="ffn",
-                    help="ffn: BASELINE configs[1] (default); train: configs[3]; decode: configs[4] (linear layers of a decode step); generate: configs[4] end to end; decoder: Budurax models beside GPT-2 of equal width")
-    ap.add_argument("--decoder-sizes", default="w768,w2048,w4096", help="decoder workload: sizes to run")
+    ap.add_argument("--workload", choices=["ffn", "train", "decode", "generate", "attention", "decoder", "lutelorn"], default="ffn",
+                    help="ffn: BASELINE configs[1] (default); train: configs[3]; decode: configs[4] (linear layers of a decode step); generate: configs[4] end to end; decoder: Budurax models beside GPT-2 of equal width; lutelorn: Lutelorn models beside Budurax of equal width")
+    ap.add_argument("--decoder-sizes", default="w768,w2048,w4096", help="decoder and lutelorn workloads: sizes to run")
     ap.add_argument("--global-batch", type=int, default=64, help="sequences per step over all GPUs (train workload); sequences of the attention workload")
     ap.add_argument("--m-per-gpu", type=int, default=M_PER_GPU, help="tokens per GPU (smaller for profiler captures)")
     ap.add_argument("--max-sms", type=int, default=0, help="SMs the GEMM kernels may occupy (0 = all; experiments)")
@@ -1348,7 +1397,7 @@ def main():
         run_attention(args)
     elif args.workload == "generate":
         run_generate(args)
-    elif args.workload == "decoder":
+    elif args.workload in ("decoder", "lutelorn"):
         run_decoder(args)
     else:
         run_ours(args)
