@@ -1159,7 +1159,7 @@ private:
                               entries_, row_entry_, row0);
             };
             RC_TRY(v_cols <= 64 ? split(grouped_split_kernel<8>) : split(grouped_split_kernel<16>));
-            return launch(grouped_combine_kernel, dim3(s.heads, rows), dim3(128), 0, act_, d.mix_out, o, ml, splits, proj_, d.proj_cols, s, entries_, row_entry_, row0);
+            return launch(grouped_combine_kernel, dim3(s.heads, rows), dim3(kGroupedCombineWarps * 32), size_t(kGroupedCombineWarps) * s.v_pad * sizeof(float), act_, d.mix_out, o, ml, splits, proj_, d.proj_cols, s, entries_, row_entry_, row0);
         }
     }
 

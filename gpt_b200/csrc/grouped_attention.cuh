@@ -344,42 +344,54 @@ grouped_split_kernel(float *__restrict__ part_o, float *__restrict__ part_ml, co
 
 constexpr int kGroupedMaxSplits = 128;
 
-// The ranges of one head put together, the output gate.  grid: (heads, rows)
-__global__ void __launch_bounds__(128)
+constexpr int kGroupedCombineWarps = 8;
+
+// The ranges of one head put together, the output gate: every warp adds up every eighth range.  grid: (heads, rows)
+__global__ void __launch_bounds__(kGroupedCombineWarps * 32)
 grouped_combine_kernel(__nv_bfloat16 *__restrict__ out, int ld_out, const float *__restrict__ part_o, const float *__restrict__ part_ml, int splits, const __nv_bfloat16 *__restrict__ proj,
                        long long ld, const GroupedShape s, const StepEntry *__restrict__ entries, const int *__restrict__ row_entry, int row0)
 {
-    __shared__ float weight[kGroupedMaxSplits];
+    extern __shared__ float sm[];   // [warps][v_pad]
+    const int h = blockIdx.x, row = row0 + blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     grid_dependency_wait();
     grid_dependency_launch();
-    const int h = blockIdx.x, row = row0 + blockIdx.y;
     const StepEntry e = entries[row_entry[row]];
     const int n = e.pos0 + row - e.row0 + 1, len = grouped_range(n, splits), used = (n + len - 1) / len;
     const long long at = (static_cast<long long>(blockIdx.y) * s.heads + h) * splits;
     const float *ml = part_ml + at * 2, *po = part_o + at * s.v_pad;
-    if (threadIdx.x < 32) {
-        float top = -FLT_MAX, sum = 0.0f;
-        for (int i = threadIdx.x; i < used; i += 32) top = fmaxf(top, ml[2 * i]);
+    float m[kGroupedMaxSplits / 32], l[kGroupedMaxSplits / 32], sum = 0.0f;
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
-        for (int i = threadIdx.x; i < used; i += 32) {
-            const float f = expf(ml[2 * i] - top);
-            weight[i] = f;
-            sum = fmaf(ml[2 * i + 1], f, sum);
+    for (int i = 0; i < kGroupedMaxSplits / 32; ++i) {
+        const float2 x = lane + 32 * i < used ? *reinterpret_cast<const float2 *>(ml + 2 * (lane + 32 * i)) : make_float2(-FLT_MAX, 0.0f);
+        m[i] = x.x;
+        l[i] = x.y;
+    }
+    float all = m[0];
+#pragma unroll
+    for (int i = 1; i < kGroupedMaxSplits / 32; ++i) all = fmaxf(all, m[i]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) all = fmaxf(all, __shfl_xor_sync(0xffffffffu, all, o));
+#pragma unroll
+    for (int i = 0; i < kGroupedMaxSplits / 32; ++i) sum = fmaf(l[i], expf(m[i] - all), sum);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    for (int c = 4 * lane; c < s.v_pad; c += 128) {
+        float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 4
+        for (int i = warp; i < used; i += kGroupedCombineWarps) {
+            const float4 v = load4(po + static_cast<long long>(i) * s.v_pad + c);
+            const float w = expf(ml[2 * i] - all);
+            acc.x = fmaf(v.x, w, acc.x); acc.y = fmaf(v.y, w, acc.y); acc.z = fmaf(v.z, w, acc.z); acc.w = fmaf(v.w, w, acc.w);
         }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        __syncwarp();
-        for (int i = threadIdx.x; i < used; i += 32) weight[i] /= sum;
+        store4(sm + warp * s.v_pad + c, acc);
     }
     __syncthreads();
     const __nv_bfloat16 *gate = proj + row * ld + s.off_g + h * s.vdim;
     for (int j = threadIdx.x; j < s.vdim; j += blockDim.x) {
-        const float g = to_f(gate[j]);
         float v = 0.0f;
-#pragma unroll 8
-        for (int i = 0; i < used; ++i) v = fmaf(po[static_cast<long long>(i) * s.v_pad + j], weight[i], v);
-        out[static_cast<long long>(row) * ld_out + h * s.vdim + j] = __float2bfloat16_rn(v * sigmoid_f(g));
+#pragma unroll
+        for (int w = 0; w < kGroupedCombineWarps; ++w) v += sm[w * s.v_pad + j];
+        out[static_cast<long long>(row) * ld_out + h * s.vdim + j] = __float2bfloat16_rn(v / sum * sigmoid_f(to_f(gate[j])));
     }
 }
 

@@ -14,6 +14,11 @@ namespace gptb200 {
 namespace dec {
 
 constexpr int kTokenCols = 32;   // value columns per block
+constexpr int kTokenAhead = 16;  // state values per thread in flight
+
+// Both kernels fetch the state (and weights) of their first token before griddepcontrol.wait: the state was written a whole step
+// ago, and so were the entries -- the embedding and the layer's norm lie between, and a kernel of a step starts no earlier than
+// the wait of the kernel before it.
 
 __host__ __device__ inline int lightning_smem_floats(int dim, bool keep_state) { return 2 * dim + kTokenCols + 8 * kTokenCols + (keep_state ? dim * kTokenCols : 0); }
 
@@ -30,8 +35,6 @@ lightning_tokens_kernel(float *__restrict__ y, const T *__restrict__ proj, long 
     const int h = blockIdx.x / slices, p0 = blockIdx.x % slices * kTokenCols;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float *k = sm, *q = k + N, *x = q + N, *part = x + kTokenCols;
-    grid_dependency_wait();
-    grid_dependency_launch();
     const StepEntry e = entries[blockIdx.y];
     float *state = reinterpret_cast<float *>(e.slot + s.ssm_state) + static_cast<long long>(h) * N * P + p0 + lane;
     const long long copy = static_cast<long long>(s.heads) * N * P;
@@ -40,6 +43,11 @@ lightning_tokens_kernel(float *__restrict__ y, const T *__restrict__ proj, long 
     const int mid_pitch = keep_state ? kTokenCols : P;
     const float keep = decay[h];
     const bool live = p0 + lane < P;
+    float head_start[kTokenAhead];
+#pragma unroll
+    for (int i = 0; i < kTokenAhead; ++i) head_start[i] = live && warp + 8 * i < N ? old[static_cast<long long>(warp + 8 * i) * P] : 0.0f;
+    grid_dependency_wait();
+    grid_dependency_launch();
     for (int t = 0; t < e.count; ++t) {
         const long long row = e.row0 + t;
         const T *r = proj + row * ld;
@@ -57,12 +65,12 @@ lightning_tokens_kernel(float *__restrict__ y, const T *__restrict__ proj, long 
         float acc = 0.0f;
         if (live) {
             const float v = x[lane];
-            for (int n0 = warp; n0 < N; n0 += 64) {   // eight rows in flight
-                float u[8];
+            for (int n0 = warp; n0 < N; n0 += 8 * kTokenAhead) {
+                float u[kTokenAhead];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) u[i] = n0 + 8 * i < N ? src[static_cast<long long>(n0 + 8 * i) * sp] : 0.0f;
+                for (int i = 0; i < kTokenAhead; ++i) u[i] = t == 0 && n0 == warp ? head_start[i] : n0 + 8 * i < N ? src[static_cast<long long>(n0 + 8 * i) * sp] : 0.0f;
 #pragma unroll
-                for (int i = 0; i < 8; ++i) {
+                for (int i = 0; i < kTokenAhead; ++i) {
                     const int n = n0 + 8 * i;
                     if (n < N) {
                         u[i] = fmaf(keep, u[i], k[n] * v);
@@ -94,8 +102,10 @@ struct WkvShape {
 
 __host__ __device__ inline int wkv_smem_floats(int dim, int rank, int threads, bool keep_state)
 {
-    return 5 * dim + rank + threads + (keep_state ? dim * dim : 0);
+    return 7 * dim + (rank + 7) / 8 * 8 + threads + (keep_state ? dim * dim : 0);
 }
+
+constexpr int kDecayPieces = 4;   // pieces of eight values of W2 that a thread keeps
 
 // One block per (head, entry).  w2 [heads * dim][w2_pitch], w0 / u / weight [heads * dim].
 template <typename T>
@@ -105,35 +115,59 @@ __global__ void wkv_tokens_kernel(T *__restrict__ out, int ld_out, const T *__re
     extern __shared__ float sm[];
     __shared__ float red[32];
     const int D = s.dim, h = blockIdx.x, lanes = blockDim.x / D;   // threads that share a value column (>= 1)
-    float *r = sm, *k = r + D, *v = k + D, *w = v + D, *bonus = w + D, *tanh_low = bonus + D, *part = tanh_low + s.rank, *S = part + blockDim.x;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    float *tanh_low = sm, *r = tanh_low + s.rank_pad, *k = r + D, *v = k + D, *gate = v + D, *w = gate + D, *bonus = w + D, *part = bonus + D, *S = part + blockDim.x;
     const int p = threadIdx.x % D, q = threadIdx.x / D;
+    // the decay's map: `share` neighbouring threads per key channel, eight values at a time
+    int share = 32;
+    while (share > 1 && share * D > static_cast<int>(blockDim.x)) share >>= 1;
+    const int channel = threadIdx.x / share, part_of = threadIdx.x % share;
+    const bool maps = channel < D;
+    const T *map = w2 + static_cast<long long>(h * D + (maps ? channel : 0)) * s.w2_pitch;
+    uint32_t kept[kDecayPieces][8];
+#pragma unroll
+    for (int i = 0; i < kDecayPieces; ++i)
+        if (maps && (part_of + i * share) * 8 < s.rank_pad) load8(map + (part_of + i * share) * 8, kept[i]);
+    const float offset = maps ? w0[h * D + channel] : 0.0f, norm_weight = weight[h * D + p];
     for (int i = threadIdx.x; i < D; i += blockDim.x) bonus[i] = u[h * D + i];
-    grid_dependency_wait();
-    grid_dependency_launch();
     const StepEntry e = entries[blockIdx.y];
     float *state = reinterpret_cast<float *>(e.slot + s.state) + static_cast<long long>(h) * D * D;
     const long long copy = static_cast<long long>(s.heads) * D * D;
     const float *old = state + e.parity * copy;
     float *next = state + (e.parity ^ 1) * copy, *mid = keep_state ? S : next;
+    float head_start[kTokenAhead];
+#pragma unroll
+    for (int i = 0; i < kTokenAhead; ++i) head_start[i] = q < lanes && q + i * lanes < D ? old[(q + i * lanes) * D + p] : 0.0f;
+    grid_dependency_wait();
+    grid_dependency_launch();
     for (int t = 0; t < e.count; ++t) {
         const long long row = e.row0 + t;
         const T *pr = proj + row * s.ld + h * D;
         __syncthreads();
-        for (int i = threadIdx.x; i < D; i += blockDim.x) {
-            r[i] = to_f(pr[i]);
-            k[i] = to_f(pr[s.group + i]);
-            v[i] = to_f(pr[2 * s.group + i]);
+        for (int i = threadIdx.x; i < 4 * D + s.rank_pad; i += blockDim.x) {   // r, k, v and the gate lie one behind the other in both places
+            if (i < 4 * D)
+                r[i] = to_f(pr[i / D * s.group + i % D]);
+            else
+                tanh_low[i - 4 * D] = i - 4 * D < s.rank ? tanhf(low[row * s.ld_low + i - 4 * D]) : 0.0f;
         }
-        for (int i = threadIdx.x; i < s.rank; i += blockDim.x) tanh_low[i] = tanhf(low[row * s.ld_low + i]);
         __syncthreads();
-        for (int c = warp; c < D; c += warps) {
-            const T *m = w2 + static_cast<long long>(h * D + c) * s.w2_pitch;
+        {
             float a = 0.0f;
-            for (int j = lane; j < s.rank; j += 32) a = fmaf(to_f(m[j]), tanh_low[j], a);
+            if (maps) {
+                auto add = [&](const uint32_t (&m)[8], int at) {
 #pragma unroll
-            for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
-            if (lane == 0) w[c] = expf(-expf(a + w0[h * D + c]));
+                    for (int j = 0; j < 8; ++j) a = fmaf(raw8<T>(m, j), tanh_low[at + j], a);
+                };
+#pragma unroll
+                for (int i = 0; i < kDecayPieces; ++i)
+                    if ((part_of + i * share) * 8 < s.rank_pad) add(kept[i], (part_of + i * share) * 8);
+                for (int at = (part_of + kDecayPieces * share) * 8; at < s.rank_pad; at += share * 8) {
+                    uint32_t m[8];
+                    load8(map + at, m);
+                    add(m, at);
+                }
+            }
+            for (int o = share >> 1; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+            if (maps && part_of == 0) w[channel] = expf(-expf(a + offset));
         }
         __syncthreads();
         const float *src = (t == 0 ? old : mid) + p;
@@ -141,12 +175,12 @@ __global__ void wkv_tokens_kernel(T *__restrict__ out, int ld_out, const T *__re
         float acc = 0.0f;
         if (q < lanes) {
             const float x = v[p];
-            for (int n0 = q; n0 < D; n0 += 8 * lanes) {   // eight rows in flight
-                float a[8];
+            for (int n0 = q; n0 < D; n0 += kTokenAhead * lanes) {
+                float a[kTokenAhead];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) a[i] = n0 + i * lanes < D ? src[(n0 + i * lanes) * D] : 0.0f;
+                for (int i = 0; i < kTokenAhead; ++i) a[i] = t == 0 && n0 == q ? head_start[i] : n0 + i * lanes < D ? src[(n0 + i * lanes) * D] : 0.0f;
 #pragma unroll
-                for (int i = 0; i < 8; ++i) {
+                for (int i = 0; i < kTokenAhead; ++i) {
                     const int n = n0 + i * lanes;
                     if (n < D) {
                         const float kv = k[n] * x;
@@ -162,7 +196,7 @@ __global__ void wkv_tokens_kernel(T *__restrict__ out, int ld_out, const T *__re
         if (q == 0)
             for (int i = 0; i < lanes; ++i) o += part[i * D + p];
         const float inv = rsqrtf(block_sum(o * o, red) / D + eps);
-        if (q == 0) out[row * ld_out + h * D + p] = from_f<T>(o * inv * weight[h * D + p] * silu_f(to_f(pr[3 * s.group + p])));
+        if (q == 0) out[row * ld_out + h * D + p] = from_f<T>(o * inv * norm_weight * silu_f(gate[p]));
     }
 }
 
