@@ -32,7 +32,7 @@ struct PrefillParams {
     int v_col0;                // first value column of head 0 in the rows of keys and values
     int rot_col0;              // shared key part in its rows
     float scale_log2;          // scale * log2(e)
-    float cap_log2, cap_in;    // CAPPED: cap * log2(e), 2 * scale / cap * log2(e)
+    float cap_log2, cap_arg;   // CAPPED: cap * log2(e), scale / cap
     __nv_bfloat16 *out;        // [rows][ld_out], head h at h * vdim
     int ld_out;
     const __nv_bfloat16 *gate; // [rows][ld_gate], head h at h * vdim
@@ -77,6 +77,16 @@ __device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t (&v
         : "memory");
 }
 
+__device__ __forceinline__ void tmem_st_32x16(uint32_t taddr, const uint32_t (&v)[16])
+{
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
+        :
+        : "r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]), "r"(v[9]), "r"(v[10]), "r"(v[11]), "r"(v[12]),
+          "r"(v[13]), "r"(v[14]), "r"(v[15])
+        : "memory");
+}
+
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
 __device__ __forceinline__ float exp2_approx(float x)
@@ -86,6 +96,47 @@ __device__ __forceinline__ float exp2_approx(float x)
     return y;
 }
 
+// two floats in one register pair
+__device__ __forceinline__ uint64_t pack2(float a, float b)
+{
+    uint64_t v;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b));
+    return v;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float &a, float &b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b)
+{
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c)
+{
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b)
+{
+    uint64_t d;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+
+// tanh of two values within [-1, 1]: x times a polynomial in x^2, the Chebyshev fit of degree 7 of tanh(x) / x (largest error 5e-9,
+// with fp32 rounding 7e-8).
+__device__ __forceinline__ uint64_t tanh_inner2(uint64_t x)
+{
+    constexpr float c[8] = {1.0f, -0.33333307504653931f, 0.13332527875900269f, -0.053887963294982910f, 0.021501919254660606f, -0.0079579148441553116f, 0.0023032133467495441f,
+                            -0.00035729847149923444f};
+    const uint64_t u = mul2(x, x);
+    uint64_t p = pack2(c[7], c[7]);
+#pragma unroll
+    for (int i = 6; i >= 0; --i) p = fma2(p, u, pack2(c[i], c[i]));
+    return mul2(p, x);
+}
+
 __device__ __forceinline__ float rcp_approx(float x)
 {
     float y;
@@ -93,10 +144,14 @@ __device__ __forceinline__ float rcp_approx(float x)
     return y;
 }
 
+// cap * tanh(x): cap - 2 cap / (1 + exp(2 x))
+__device__ __forceinline__ float capped(float x, float cap) { return fmaf(-2.0f * cap, rcp_approx(1.0f + exp2_approx(x * 2.8853900817779268f)), cap); }
+
 }  // namespace ptx_attn
 
-// map_kv: rows of [keys of all heads | values of all heads]; map_shared: rows with the key part that all heads share.
-// CAPPED: scores become cap * tanh(score / cap), in the form cap - 2 cap / (1 + exp(2 score / cap)).
+// grid: (heads, blocks of 256 rows).  map_kv: rows of [keys of all heads | values of all heads]; map_shared: rows with the key part that all heads share.
+// CAPPED: scores become cap * tanh(score / cap).  Special-function instructions (exponential, reciprocal) are what this kernel runs out of
+// first, so where all scores of a warp's rows lie within the cap tanh is a polynomial; else 1 - 2 / (1 + exp(2 score / cap)).
 template <bool CAPPED>
 __global__ void __launch_bounds__(kPrefillThreads, 1)
 attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_shared, const PrefillParams p)
@@ -122,8 +177,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     volatile uint32_t *abort_flag = tmem_slot + 1;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int head = blockIdx.y, kv_head = head / p.kv_share;
-    const int row_base = (gridDim.x - 1 - blockIdx.x) * 256;   // the longest rows first
+    const int head = blockIdx.x, kv_head = head / p.kv_share;
+    const int row_base = (gridDim.y - 1 - blockIdx.y) * 256;   // the longest rows of all heads first
     // key blocks of the two tiles
     int n_blocks[2];
 #pragma unroll
@@ -214,7 +269,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 for (int part = 0; part < 2; ++part)
                     for (int k = 0; k < 8; ++k) {
                         const uint64_t db = ptx::make_smem_desc(va + k * 2048, kPrefillBlock, 1024, ptx::kLayoutSw128);
-                        ptx_attn::mma_f16_ts(tmem + 256 + 128 * g, tmem + 128 * g + 64 * part + 8 * k, db, idesc_o, acc);
+                        ptx_attn::mma_f16_ts(tmem + 256 + 128 * g, tmem + 128 * g + 32 * (k >> 1) + 8 * (k & 1) + 16 * part, db, idesc_o, acc);
                         acc = 1;
                     }
                 if (j + 1 == n_blocks[g]) ptx::mma_commit(o_full(g));
@@ -260,30 +315,43 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         for (int j = 0; j < blocks; ++j) {
             if (!bounded_wait(s_full(g), j & 1, abort_flag, p.status, DEV_TIMEOUT_EPILOGUE)) { ok = false; break; }
             ptx::tc_fence_after();
-            float s[128];
+            const bool whole = j * 128 + 127 <= p.pos0 + row_base + g * 128;   // the tile's first row sees all of this block
+            const int seen = last - j * 128;                                   // this row: keys 0 .. seen of the block
+            // 1. the row's largest score
+            bool near_zero = true;   // no score of the warp's rows beyond the cap: tanh is a polynomial
+            float top;
+            {
+                float most[4] = {-FLT_MAX, -FLT_MAX, -FLT_MAX, -FLT_MAX}, widest[4] = {};
+                uint32_t r[2][32];
+                ptx::tmem_ld_32x32(s_addr, r[0]);
 #pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                uint32_t r[32];
-                ptx::tmem_ld_32x32(s_addr + 32 * c, r);
-                ptx::tmem_ld_wait();
+                for (int c = 0; c < 4; ++c) {
+                    ptx::tmem_ld_wait();
+                    if (c < 3) ptx::tmem_ld_32x32(s_addr + 32 * (c + 1), r[(c + 1) & 1]);
+                    if (CAPPED) {
 #pragma unroll
-                for (int i = 0; i < 32; ++i) {
-                    const float x = __uint_as_float(r[i]);
-                    s[32 * c + i] = CAPPED ? fmaf(-2.0f * p.cap_log2, ptx_attn::rcp_approx(1.0f + ptx_attn::exp2_approx(x * p.cap_in)), p.cap_log2) : x * p.scale_log2;
+                        for (int i = 0; i < 32; ++i) widest[i & 3] = fmaxf(widest[i & 3], fabsf(__uint_as_float(r[c & 1][i])));
+                    }
+                    if (whole) {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i) most[i & 3] = fmaxf(most[i & 3], __uint_as_float(r[c & 1][i]));
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i) most[i & 3] = fmaxf(most[i & 3], 32 * c + i <= seen ? __uint_as_float(r[c & 1][i]) : -FLT_MAX);
+                    }
+                }
+                top = fmaxf(fmaxf(most[0], most[1]), fmaxf(most[2], most[3]));
+                if (CAPPED) {
+                    near_zero = __all_sync(0xffffffffu, fmaxf(fmaxf(widest[0], widest[1]), fmaxf(widest[2], widest[3])) * p.cap_arg <= 1.0f);
+                    top = ptx_attn::capped(fmaxf(top, -1e30f) * p.cap_arg, p.cap_log2);
+                } else {
+                    top = fmaxf(top, -1e30f) * p.scale_log2;
                 }
             }
-            if (j * 128 + 127 > p.pos0 + row_base + g * 128) {   // the tile's first row does not see all of this block
-#pragma unroll
-                for (int i = 0; i < 128; ++i)
-                    if (j * 128 + i > last) s[i] = -FLT_MAX;
-            }
-            float top = s[0];
-#pragma unroll
-            for (int i = 1; i < 128; ++i) top = fmaxf(top, s[i]);
             if (j == 0) {
                 ref = top;   // key 0 is visible to every row
             } else {
-                const bool grow = top > ref + 8.0f;
+                const bool grow = top > ref + 8.0f;   // never where the row sees nothing of this block
                 if (__any_sync(0xffffffffu, grow)) {
                     // earlier weights refer to the old maximum: scale O (complete: this block's scores come after it) and the sum
                     const float f = grow ? ptx_attn::exp2_approx(ref - top) : 1.0f;
@@ -299,27 +367,46 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                     }
                 }
             }
-            uint32_t hi[64];
+            // 2. the weights: 32 at a time they take the place of their scores, 16 columns of first terms, 16 of second terms
+            const uint64_t scale2 = ptx_attn::pack2(CAPPED ? p.cap_arg : p.scale_log2, CAPPED ? p.cap_arg : p.scale_log2), cap2 = ptx_attn::pack2(p.cap_log2, p.cap_log2),
+                           minus_ref = ptx_attn::pack2(-ref, -ref);
+            uint64_t sums[2] = {0, 0};
+#pragma unroll 1
+            for (int c = 0; c < 4; ++c) {
+                uint32_t r[32], hi[16], lo[16];
+                ptx::tmem_ld_32x32(s_addr + 32 * c, r);
+                ptx::tmem_ld_wait();
+                float x[32];
+                if (!CAPPED || near_zero) {
 #pragma unroll
-            for (int i = 0; i < 64; ++i) {
-                const float a = ptx_attn::exp2_approx(s[2 * i] - ref), b = ptx_attn::exp2_approx(s[2 * i + 1] - ref);
+                    for (int i = 0; i < 32; i += 2) {
+                        const uint64_t v = ptx_attn::pack2(__uint_as_float(r[i]), __uint_as_float(r[i + 1]));
+                        ptx_attn::unpack2(CAPPED ? ptx_attn::fma2(ptx_attn::tanh_inner2(ptx_attn::mul2(v, scale2)), cap2, minus_ref) : ptx_attn::fma2(v, scale2, minus_ref), x[i], x[i + 1]);
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) x[i] = ptx_attn::capped(__uint_as_float(r[i]) * p.cap_arg, p.cap_log2) - ref;
+                }
+                if (!whole) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i)
+                        if (32 * c + i > seen) x[i] = -1e30f;
+                }
+#pragma unroll
+                for (int i = 0; i < 16; ++i) {
+                    const float a = ptx_attn::exp2_approx(x[2 * i]), b = ptx_attn::exp2_approx(x[2 * i + 1]);
+                    const uint64_t v = ptx_attn::pack2(a, b);
+                    sums[i & 1] = ptx_attn::add2(sums[i & 1], v);
+                    hi[i] = ptx::pack_bf16x2(a, b);
+                    lo[i] = ptx::pack_bf16x2(a - bf16_lo(hi[i]), b - bf16_hi(hi[i]));
+                }
+                ptx_attn::tmem_st_32x16(s_addr + 32 * c, hi);
+                ptx_attn::tmem_st_32x16(s_addr + 32 * c + 16, lo);
+            }
+            {
+                float a, b;
+                ptx_attn::unpack2(ptx_attn::add2(sums[0], sums[1]), a, b);
                 sum += a + b;
-                hi[i] = ptx::pack_bf16x2(a, b);
-                s[i] = __uint_as_float(ptx::pack_bf16x2(a - bf16_lo(hi[i]), b - bf16_hi(hi[i])));   // second terms, in the values already used
-            }
-#pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                uint32_t r[32];
-#pragma unroll
-                for (int i = 0; i < 32; ++i) r[i] = hi[32 * c + i];
-                ptx_attn::tmem_st_32x32(s_addr + 32 * c, r);
-            }
-#pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                uint32_t r[32];
-#pragma unroll
-                for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(s[32 * c + i]);
-                ptx_attn::tmem_st_32x32(s_addr + 64 + 32 * c, r);
             }
             ptx_attn::tmem_st_wait();
             ptx::tc_fence_before();

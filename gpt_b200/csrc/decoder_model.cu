@@ -280,8 +280,8 @@ public:
             segment_tokens_ = value;
             return GPTB200_OK;
         }
-        if (!strcmp(key, "wkv_segment_tokens")) {   // wkv prompts: tokens per segment (a multiple of 16)
-            if (value < kWkvChunk || value % kWkvChunk) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "wkv_segment_tokens must be a multiple of %d", kWkvChunk);
+        if (!strcmp(key, "wkv_segment_tokens")) {   // wkv prompts: tokens per segment (a multiple of 16; 0: automatic)
+            if (value < 0 || value % kWkvChunk) return fail(ctx_, GPTB200_ERR_INVALID_ARG, "wkv_segment_tokens must be a multiple of %d", kWkvChunk);
             wkv_segment_tokens_ = value;
             return GPTB200_OK;
         }
@@ -1048,7 +1048,7 @@ private:
             p.out = act_ + size_t(part.row0) * d.mix_out; p.ld_out = d.mix_out;
             p.gate = q + s.off_g; p.ld_gate = d.proj_cols;
             p.status = ctx_->d_status;
-            return launch(attention_prefill_kernel<false>, dim3((part.count + 255) / 256, s.heads), dim3(kPrefillThreads),
+            return launch(attention_prefill_kernel<false>, dim3(s.heads, (part.count + 255) / 256), dim3(kPrefillThreads),
                           size_t(prefill_smem_bytes(p.u_blocks, p.r_blocks, p.v_blocks, p.k_stages, p.v_stages)), mq, mkv, mc, p);
         }
     }
@@ -1187,13 +1187,13 @@ private:
             p.scale_log2 = static_cast<float>(s.scale * kLog2e);
             if (s.softcap > 0.0f) {
                 p.cap_log2 = static_cast<float>(s.softcap * kLog2e);
-                p.cap_in = static_cast<float>(2.0 * s.scale / s.softcap * kLog2e);
+                p.cap_arg = s.scale / s.softcap;
             }
             p.out = act_ + size_t(part.row0) * d.mix_out; p.ld_out = d.mix_out;
             p.gate = q + s.off_g; p.ld_gate = d.proj_cols;
             p.status = ctx_->d_status;
             const size_t smem = size_t(prefill_smem_bytes(p.u_blocks, 0, p.v_blocks, k_stages, v_stages));
-            const dim3 grid((part.count + 255) / 256, s.heads);
+            const dim3 grid(s.heads, (part.count + 255) / 256);
             return s.softcap > 0.0f ? launch(attention_prefill_kernel<true>, grid, dim3(kPrefillThreads), smem, mq, mkv, mkv, p)
                                     : launch(attention_prefill_kernel<false>, grid, dim3(kPrefillThreads), smem, mq, mkv, mkv, p);
         }
@@ -1281,7 +1281,10 @@ private:
         } else {
             int longest = 0;
             for (int i = 0; i < n; ++i) longest = std::max(longest, parts[entry0 + i].count);
-            const int tokens = longest > wkv_segment_tokens_ + wkv_segment_tokens_ / 2 ? wkv_segment_tokens_ : pad_to(longest, kWkvChunk), segments = (longest + tokens - 1) / tokens;
+            // segments: as many blocks as fit the machine at once, none shorter than a few chunks
+            int segment = wkv_segment_tokens_;
+            if (segment == 0) segment = std::max(4 * kWkvChunk, pad_to(static_cast<int>(1LL * longest * n * s.heads / (wkv_blocks(KT) * ctx_->num_sms)), kWkvChunk));
+            const int tokens = longest > segment + segment / 2 ? segment : pad_to(longest, kWkvChunk), segments = (longest + tokens - 1) / tokens;
             const size_t smem = wkv_chunk_layout(KT).total, square = size_t(s.dim) * s.dim;
             float *seg_state = nullptr, *seg_decay = nullptr;
             const auto chunks = [&](auto kernel, int launched) {
@@ -1435,7 +1438,7 @@ private:
     size_t fixed_state_ = 0, position_bytes_ = 0, previous_state_ = 0;
     std::vector<void *> weights_, work_;
     std::vector<Slot> slots_;
-    int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8, segment_tokens_ = 1024, wkv_segment_tokens_ = 256;
+    int pass_rows_ = 4096, expand_rows_ = 32, chunk_rows_ = 8, segment_tokens_ = 1024, wkv_segment_tokens_ = 0;
     T *expanded_ = nullptr;
     size_t expanded_count_ = 0;
     float *scratch_ = nullptr;

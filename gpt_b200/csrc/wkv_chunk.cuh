@@ -25,6 +25,9 @@ namespace dec {
 constexpr int kWkvChunk = 16;
 constexpr int kWkvMaxDim = 128;
 
+// blocks per SM that registers and shared memory allow
+__host__ __device__ constexpr int wkv_blocks(int kt) { return kt == 8 ? 2 : kt == 4 ? 4 : 8; }
+
 struct WkvChunkLayout {
     int xp, fp;                     // row pitches of bf16 tiles (bytes) and fp32 tiles (floats)
     int tile, raw, buf;             // bytes: bf16 tile, offset of the fp32 tile in a buffer, one buffer
@@ -70,7 +73,7 @@ __global__ void wkv_low_rank_kernel(__nv_bfloat16 *__restrict__ out, int rank_pa
 // KT: tiles of 16 channels (heads of up to 16 * KT), one warp each.  raw [rows][ld_raw]: W2 tanh(W1 x).  segment_state
 // [entry][head][segment][dim][dim], segment_decay [entry][head][segment][dim].  grid: (heads, entries, segments)
 template <int KT, bool SEGMENT_STATES>
-__global__ void __launch_bounds__(32 * KT, KT == 8 ? 2 : KT == 4 ? 4 : 8)
+__global__ void __launch_bounds__(32 * KT, wkv_blocks(KT))
 wkv_chunk_kernel(__nv_bfloat16 *__restrict__ out, int ld_out, const __nv_bfloat16 *__restrict__ proj, const float *__restrict__ raw, int ld_raw, const float *__restrict__ w0,
                  const float *__restrict__ bonus, const float *__restrict__ weight, float eps, const WkvShape s, const StepEntry *__restrict__ entries, int segment_tokens, int max_segments,
                  float *__restrict__ segment_state, float *__restrict__ segment_decay)
