@@ -336,9 +336,12 @@ int gptb200_model_load_state(gptb200_model *m, const char *path);
 int gptb200_model_step_count(gptb200_model *m);
 
 /* ---- decoder models described by a folder with config.json and model.safetensors (no counterpart in the reference, whose one
- *      model is GPT-2).  config.json names the architecture ("Budurax": Mamba-2 and latent-attention layers in any order, gated
- *      GELU feed-forwards, layer norms before and after each sublayer, token shift, per-layer token input, depth average) and gives
- *      every size and constant; gptb200_decoder_load chooses the model class by it.
+ *      model is GPT-2).  config.json names the architecture and gives every size and constant; gptb200_decoder_load chooses the model
+ *      class by it.  "Budurax": gated GELU feed-forwards, layer norms before and after each sublayer, token shift, per-layer token
+ *      input, depth average.  "Lutelorn": gated SiLU feed-forwards, RMS norms before the sublayers, a residual multiplier, an
+ *      embedding of the pair (previous token, token).  Layers, in any order: "mamba2", "latent_attention", "attention" (grouped heads, biases,
+ *      rotated neighbours, capped scores, values blended with the first layer's, output gate), "lightning" (linear attention with
+ *      constant decays), "wkv" (linear attention with a decay per channel and token; Lutelorn only).
  *   dtype           GPTB200_DTYPE_BF16: weights, activations and caches in bf16, products on the tensor cores (up to eight rows:
  *                   streamed weights) with fp32 accumulation; residual stream, norms, softmax and recurrences in fp32.
  *                   GPTB200_DTYPE_F32: everything in fp32 FMAs.
@@ -350,10 +353,12 @@ int gptb200_model_step_count(gptb200_model *m);
  *                   the device: temperature 0 takes the largest logit, otherwise a draw from softmax(logits / temperature).  The
  *                   last sampled token is not run.
  *   message         receives the reason when loading fails (capacity bytes); later errors: gptb200_last_error(context).
- *   options         "pass_rows" (most rows of one pass of a step, default 4096), "expand_rows" (latent attention in bf16: shortest portion
- *                   whose keys and values are expanded for the tensor cores, default 32; shorter ones use the latents as they are),
- *                   "chunk_rows" (Mamba-2 in bf16: shortest portion that runs in chunks on the tensor cores, default 8; shorter ones token by
- *                   token), "segment_tokens" (Mamba-2 prompts: tokens per segment of the segments that run side by side, default 1024) and those of gptb200_ctx_set_option */
+ *   options         "pass_rows" (most rows of one pass of a step, default 4096), "expand_rows" (attention in bf16: shortest portion that runs
+ *                   in the tensor-core form for prompts, default 32; shorter ones split the positions, latent attention then uses the
+ *                   latents as they are), "chunk_rows" (recurrent layers in bf16: shortest portion that runs in chunks on the tensor
+ *                   cores, default 8; shorter ones token by token), "segment_tokens" (Mamba-2 and lightning prompts: tokens per segment of the
+ *                   segments that run side by side, default 1024), "wkv_segment_tokens" (the same for wkv, a multiple of 16, default 0:
+ *                   automatic) and those of gptb200_ctx_set_option */
 typedef enum gptb200_dtype { GPTB200_DTYPE_BF16 = 0, GPTB200_DTYPE_F32 = 1 } gptb200_dtype;
 typedef struct gptb200_decoder gptb200_decoder;
 int gptb200_decoder_check_config(const char *config_json, char *message, size_t capacity);   /* host only */
@@ -375,6 +380,7 @@ int gptb200_rotary_frequencies(int dims, double base, const double *scaling4, do
  *   kind 0  out fp32
  *        1  out bf16; columns from tail_col (a multiple of 32; n or more: none) on stay fp32 and go to tail [m x tail_pitch]
  *        2  gated: columns of w come in groups of 32 gate | 32 up (n a multiple of 64), out bf16 [m x n/2] = gelu_tanh(gate) * up
+ *        4  as 2 with silu(gate) * up
  *        3  out bf16 = gelu_tanh(product) * factor[factor_rows[row]][column], factor bf16 with row pitch factor_pitch (n a multiple of 8)
  * Up to 8 rows (option "gemv_rows") a weight-streaming kernel, else the tcgen05 kernels. */
 int gptb200_linear_bf16(gptb200_ctx *ctx, int kind, void *out, long long out_pitch, const void *x, long long x_pitch, const void *w, int m, int n, int k, float *tail,

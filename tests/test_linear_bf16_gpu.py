@@ -71,6 +71,10 @@ def test_forms(backend, m, n, k):
     run(backend, 2, out, x, w, n)
     close(out[:m, :n // 2], (gelu(g[:, :, 0]) * g[:, :, 1]).reshape(m, n // 2), 5e-3)
     assert (out[:, n // 2:] == 77).all() and (out[m] == 77).all()
+    out = guard(m, n // 2 + 8, torch.bfloat16)
+    run(backend, 4, out, x, w, n)
+    close(out[:m, :n // 2], (torch.nn.functional.silu(g[:, :, 0]) * g[:, :, 1]).reshape(m, n // 2), 5e-3)
+    assert (out[:, n // 2:] == 77).all() and (out[m] == 77).all()
     factor = torch.randn(13, n + 8, device="cuda").bfloat16()
     rows = torch.randint(0, 13, (m,), device="cuda", dtype=torch.int32)
     out = guard(m, n + 8, torch.bfloat16)
@@ -107,5 +111,6 @@ def test_wrong_sizes_are_refused(backend):
     assert lib.gptb200_linear_bf16(*args(0, 64, 60, 64)) == 1       # k not a multiple of 8
     assert lib.gptb200_linear_bf16(*args(0, 64, 64, 60)) == 1       # pitch
     assert lib.gptb200_linear_bf16(*args(2, 96, 64, 64)) == 1       # gated columns
+    assert lib.gptb200_linear_bf16(*args(4, 96, 64, 64)) == 1
     assert lib.gptb200_linear_bf16(*args(3, 64, 64, 64)) == 1       # no factor
     assert lib.gptb200_linear_bf16(*args(7, 64, 64, 64)) == 1       # kind

@@ -124,10 +124,11 @@ def test_wide_layers_on_every_product_kernel(tmp_path, dtype):
     tokens = np.random.default_rng(21).integers(0, c["vocab"], 330)
     want = lutelorn.forward(c, w, tokens)
     model = load(tmp_path, c, w, dtype)
-    for pair in (0, 1, -1):
-        model.set_option("pair", pair)
+    for option, value in (("pair", 0), ("pair", 1), ("pair", -1), ("stream_k", 1), ("tile_n", 128)):
+        model.set_option("pair", 0)
+        model.set_option(option, value)
         for cuts in (PROMPT, (200, 33, 90, 5, 1)):
-            assert dm.close(whole(model, tokens, cuts), want, TOL[dtype]), (pair, cuts)
+            assert dm.close(whole(model, tokens, cuts), want, TOL[dtype]), (option, value, cuts)
     model.close_model()
 
 
